@@ -45,6 +45,10 @@ typedef void* umbs_stream_t; /* cudaStream_t */
 #define UMBS_MIX_MLSTM 3             /* matrix memory with exponential gates and a running maximum */
 #define UMBS_MIX_TIME_MIX 4          /* matrix memory with a decay per key channel and token, computed from the token itself;
                                       * five token-shifted mixes of the input feed its projections */
+#define UMBS_MIX_GATED_DELTA 5       /* matrix memory written by the delta rule (what it already returns for the key is taken off the
+                                      * value), one decay per head and token; short convolution on q, k and v, unit q and k */
+#define UMBS_MIX_SSD 6               /* state-space memory: one decay and one step size per head and token, input and read-out vectors
+                                      * shared by groups of heads, a skip per head, short convolution in front, gate before the norm */
 
 /* How a layer is put together.  PARALLEL: one group norm feeds the mixer (token-shifted) and the feed-forward side by
  * side, the sum goes through the depth average.  PRENORM: x += mixer(norm1(x)), then x += ff(norm2(x)). */
@@ -71,6 +75,10 @@ typedef void* umbs_stream_t; /* cudaStream_t */
                                       * scores the sum of its two largest scores, only experts of the `keep` best groups are
                                       * eligible; the `top` largest eligible scores, divided by their sum (+ 1e-20) */
 #define UMBS_ROUTE_SOFTMAX_ALL 2     /* softmax over all experts; the `top` largest scores, as they are (not renormalised) */
+
+/* What a rank-one memory writes (umbs_memory_t.rule): S <- decay S + k u^T with */
+#define UMBS_MEMORY_ADD 0            /* u = strength v */
+#define UMBS_MEMORY_DELTA 1          /* u = strength (v - (decay S)^T k) */
 
 /* How attention turns scores into weights. */
 #define UMBS_ATTN_SOFTMAX 0          /* p = exp(s) / sum exp(s) */
@@ -220,6 +228,22 @@ typedef struct umbs_layer_s {
      * mix_scale * first + second_scale * second.  Only its mixer fields are read (no norms, no feed-forward). */
     const struct umbs_layer_s* second;
     float mix_scale, second_scale;      /* read only with a second mixer */
+    /* pre-norm form: norms behind the blocks, x += rms_norm(block output) * w (eps of the model) */
+    const float* post_norm_w;  /* fp32 [width] or NULL: behind the mixer */
+    const float* post_norm2_w; /* the same behind the feed-forward */
+    /* pre-norm form: in front of this layer x <- w_merge [x; x0], x0 the embedding output; [width, 2 width] or NULL */
+    const void* w_merge;
+    /* gated delta rule and state-space memory (use heads, kv_heads (query / key heads; groups), dim (= state size), vdim, taps,
+     * conv_w (fp32 [2 kv_heads dim + heads vdim, taps]), conv_state (fp32 [2, slots, taps - 1, the same channels]), out_norm_w
+     * (gated delta: fp32 [vdim]; state space: fp32 [heads vdim])).  w_in rows, gated delta: q | k | v | gate (heads vdim) |
+     * write strength (heads) | decay input (heads); state space: gate (heads vdim) | v (heads vdim) | k (kv_heads dim) |
+     * q (kv_heads dim) | step size (heads). */
+    const float* conv_b;       /* fp32 [channels] or NULL: bias of the convolution */
+    const float* decay_rate;   /* fp32 [heads]: decay = exp(-decay_rate softplus(decay input + dt_bias)) */
+    const float* dt_bias;      /* fp32 [heads] */
+    const float* skip_w;       /* fp32 [heads] or NULL: o += skip v */
+    int norm_parts;            /* state space: equal parts of the output that are normed on their own */
+    float* mem_state;          /* fp32 [slots, heads, vdim, dim]: key index last */
 } umbs_layer_t;
 
 typedef struct {
@@ -238,6 +262,7 @@ typedef struct {
     float final_norm_alpha;    /* UMBS_NORM_DYT */
     const float* pos_freq;     /* fp32 [width / 2] or NULL: sinusoidal positions are added to the embedding,
                                 * entry 2i += sin(position pos_freq[i]), entry 2i + 1 += cos(position pos_freq[i]) */
+    const float* embed_norm;   /* fp32 [width] or NULL: the embedding row is RMS-normed with this weight (goes with no pos_freq) */
 } umbs_model_t;
 
 const char* umbs_version(void);
@@ -395,6 +420,7 @@ typedef struct {
     float delta_mult;          /* factor on delta alone (with delta2 == NULL, 0 reads as 1) */
     const float* delta2;       /* fp32 [n, width] or NULL: a second dense part, added as delta2_mult * delta2 */
     float delta2_mult;
+    const float* norm_w;       /* fp32 [width] or NULL: the sum is RMS-normed with this weight (the call's eps) before scale and mult */
 } umbs_delta_t;
 
 /* umbs_add_rms_norm for any pending output and either norm: x[t] += pending(t) (d may be NULL), copy, and
@@ -407,6 +433,16 @@ int umbs_add_norm(int dtype, float* x, const umbs_delta_t* d, const int32_t* row
 int umbs_add_norm_ex(int dtype, float* x, const umbs_delta_t* d, const int32_t* rows, int n, int kind, const float* w,
                      const float* b, float w_offset, float alpha, int width, float eps, void* y, float* copy,
                      umbs_stream_t stream);
+
+/* y[t] = x[t] + pending(t) as `dtype`, row stride ldy (x is updated, copy as in umbs_add_norm): the rows of a matrix product
+ * that reads the residual stream itself.  eps: of the pending output's own norm. */
+int umbs_add_rows(int dtype, float* x, const umbs_delta_t* d, int n, int width, float eps, void* y, int64_t ldy, float* copy,
+                  umbs_stream_t stream);
+
+/* Embedding row through an RMS norm: y[t] = r / sqrt(mean(r^2) + eps) * w with r = table[ids[t]] * scale (fp32), and the same as
+ * `dtype` in y2 (row stride ld2) unless it is NULL. */
+int umbs_embedding_norm(int dtype, const int32_t* ids, const void* table, float scale, const float* w, float eps, float* y, void* y2,
+                        int64_t ld2, int n, int width, umbs_stream_t stream);
 
 /* z <- cap tanh(z / cap), fp32, n values. */
 int umbs_softcap(float* z, int64_t n, float cap, umbs_stream_t stream);
@@ -510,6 +546,46 @@ int umbs_shift_mix(int dtype, const void* h, const float* mu, int n_mix, float* 
 int umbs_time_mix(int dtype, const float* proj, int64_t ld, const float* decay_raw, const float* decay_bias,
                   const float* bonus, const umbs_batch_t* batch, int heads, int dim, float eps, const float* out_norm_w,
                   float* state, float* o_scratch, void* out, umbs_stream_t stream);
+
+/* ---- rank-one memories: the gated delta rule, state-space layers ----
+ *
+ * Per head, with a decay and a write strength per token: S <- decay S + k u^T (u by `rule`), o = S^T q (+ skip v), the read-out
+ * seeing the current token's write.  The state S is dim x vdim, stored fp32 [slots, heads, vdim, dim] (key index last), read as
+ * zero at position 0.  Head h reads the query / key head h / (heads / kv_heads). */
+typedef struct {
+    int rule;                  /* UMBS_MEMORY_* */
+    int heads, kv_heads, dim, vdim;      /* dim <= 512 */
+    /* short causal convolution (then silu) over the channels q, k, v of the projection; channel c is its column off_conv + c */
+    int taps;                  /* last tap = the current token */
+    int off_conv, off_q, off_k, off_v;   /* off_q, off_k, off_v: first channel of the queries, keys and values */
+    const float* conv_w;       /* fp32 [channels, taps], channels = 2 kv_heads dim + heads vdim */
+    const float* conv_b;       /* fp32 [channels] or NULL */
+    float* conv_state;         /* fp32 [2, slots, taps - 1, channels], double-buffered by the sequence's parity (NULL with one tap) */
+    int unit;                  /* q and k become unit vectors per head (x / sqrt(sum x^2 + 1e-6)), q also times dim^-1/2 */
+    /* decay = exp(-decay_rate softplus(z + dt_bias)), z = column off_decay + head of the projection; strength = sigmoid of column
+     * off_strength + head, or (off_strength < 0) the step size softplus(z + dt_bias) itself */
+    int off_decay, off_strength;
+    const float* decay_rate;   /* fp32 [heads] */
+    const float* dt_bias;      /* fp32 [heads] */
+    const float* skip;         /* fp32 [heads] or NULL */
+    float* state;
+} umbs_memory_t;
+
+/* What stands between the in-projection (fp32 [n_tokens, ld]) and the recurrence: convolution, silu, unit norms, gates.
+ * qkv: fp32 [n_tokens, ld_qkv], the channels as the recurrence reads them; gates: fp32 [n_tokens, heads, 2] = logarithm of the
+ * decay, strength; kq: fp32 [n_tokens, kv_heads] = k . q. */
+int umbs_memory_prep(const float* proj, int64_t ld, const umbs_memory_t* mem, const umbs_batch_t* batch, int slots, float* qkv,
+                     int64_t ld_qkv, float* gates, float* kq, umbs_stream_t stream);
+
+/* The recurrence over what umbs_memory_prep left.  o: fp32 [n_tokens, heads vdim]. */
+int umbs_memory_run(const float* qkv, int64_t ld_qkv, const float* gates, const float* kq, const umbs_memory_t* mem,
+                    const umbs_batch_t* batch, float* o, umbs_stream_t stream);
+
+/* Gated unit norm of every one of `parts` equal parts of a row of o (fp32 [n, width]): with gate_first
+ * out = unit(o silu(gate)) * w, else out = unit(o) * w * silu(gate); unit(y) = y / sqrt(mean(y^2) + eps) over the part.
+ * gate: fp32, row stride ldg; w: fp32 [w_len], element e of a row uses w[e mod w_len].  out: `dtype` [n, width]. */
+int umbs_gated_norm(int dtype, const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w, int w_len,
+                    int gate_first, float eps, void* out, umbs_stream_t stream);
 
 /* umbs_gemm_ex for a plain product followed by a unary activation (UMBS_UNARY_*, with its two numbers). */
 int umbs_gemm_unary(int dtype, const void* A, int64_t lda, int a_goff, const void* W, int64_t ldw, int64_t w_gstride, void* C,

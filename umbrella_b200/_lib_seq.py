@@ -1,7 +1,7 @@
 """ctypes binding of libumbrella_b200_seq.so (the C ABI declared in include/umbrella_b200_seq.h): the batched step
 of the sequence-state decoders and its building blocks.
 
-The library is compiled in-tree on first use when it is missing or older than its sources (``build.build_seq``: eight
+The library is compiled in-tree on first use when it is missing or older than its sources (``build.build_seq``: nine
 small translation units, seconds) -- a fresh checkout serves these models without a separate build step.  There is
 no PyTorch / CPU fallback behind these calls: without nvcc and without the library, loading is an error.
 """
@@ -17,6 +17,8 @@ LIB_PATH = os.path.join(HERE, "libumbrella_b200_seq.so")
 
 UMBS_BF16, UMBS_F32 = 0, 1
 UMBS_MIX_RETENTION, UMBS_MIX_LATENT_ATTENTION, UMBS_MIX_CACHED_ATTENTION, UMBS_MIX_MLSTM, UMBS_MIX_TIME_MIX = 0, 1, 2, 3, 4
+UMBS_MIX_GATED_DELTA, UMBS_MIX_SSD = 5, 6
+UMBS_MEMORY_ADD, UMBS_MEMORY_DELTA = 0, 1
 UMBS_FORM_PARALLEL, UMBS_FORM_PRENORM = 0, 1
 UMBS_ACT_CLAMPED_GLU, UMBS_ACT_GELU_TANH, UMBS_ACT_SILU = 1, 2, 3
 UMBS_NORM_RMS, UMBS_NORM_LAYER, UMBS_NORM_DYT = 0, 1, 2
@@ -43,7 +45,7 @@ class Mlp(C.Structure):
 class Delta(C.Structure):
     _fields_ = [("delta", c_void_p), ("pair_out", c_void_p), ("sel_w", c_void_p), ("pair_pos", c_void_p), ("top", c_int),
                 ("shared", c_void_p), ("shared_gate", c_void_p), ("scale", c_void_p), ("mult", c_float),
-                ("delta_mult", c_float), ("delta2", c_void_p), ("delta2_mult", c_float)]
+                ("delta_mult", c_float), ("delta2", c_void_p), ("delta2_mult", c_float), ("norm_w", c_void_p)]
 
 
 class Layer(C.Structure):
@@ -69,7 +71,9 @@ Layer._fields_ = [("mixer", c_int), ("heads", c_int), ("dim", c_int), ("vdim", c
                 ("head_unit_norm", c_int), ("out_mult", c_float), ("q_norm_w", c_void_p), ("k_norm_w", c_void_p),
                 ("kv_from", c_int), ("mix_mu", c_void_p), ("decay_rank", c_int), ("w_decay1", c_void_p),
                 ("w_decay2", c_void_p), ("decay_bias", c_void_p), ("bonus", c_void_p), ("tm_state", c_void_p),
-                ("second", C.POINTER(Layer)), ("mix_scale", c_float), ("second_scale", c_float)]
+                ("second", C.POINTER(Layer)), ("mix_scale", c_float), ("second_scale", c_float),
+                ("post_norm_w", c_void_p), ("post_norm2_w", c_void_p), ("w_merge", c_void_p), ("conv_b", c_void_p),
+                ("decay_rate", c_void_p), ("dt_bias", c_void_p), ("skip_w", c_void_p), ("norm_parts", c_int), ("mem_state", c_void_p)]
 
 
 class Model(C.Structure):
@@ -77,12 +81,19 @@ class Model(C.Structure):
                 ("slots", c_int), ("norm_eps", c_float), ("embed", c_void_p), ("final_norm", c_void_p), ("head", c_void_p),
                 ("layers", C.POINTER(Layer)), ("norm_offset", c_float), ("logit_softcap", c_float),
                 ("embed_scale", c_float), ("norm_kind", c_int), ("final_norm_b", c_void_p), ("final_norm_alpha", c_float),
-                ("pos_freq", c_void_p)]
+                ("pos_freq", c_void_p), ("embed_norm", c_void_p)]
 
 
 class AttnOpts(C.Structure):
     _fields_ = [("softcap", c_float), ("dist_r1", c_void_p), ("dist_r2", c_void_p), ("chunk", c_int), ("maps", c_int),
                 ("value_heads", c_int), ("raw_out", c_void_p)]
+
+
+class Memory(C.Structure):
+    _fields_ = [("rule", c_int), ("heads", c_int), ("kv_heads", c_int), ("dim", c_int), ("vdim", c_int), ("taps", c_int),
+                ("off_conv", c_int), ("off_q", c_int), ("off_k", c_int), ("off_v", c_int), ("conv_w", c_void_p), ("conv_b", c_void_p),
+                ("conv_state", c_void_p), ("unit", c_int), ("off_decay", c_int), ("off_strength", c_int), ("decay_rate", c_void_p),
+                ("dt_bias", c_void_p), ("skip", c_void_p), ("state", c_void_p)]
 
 
 _BP = C.POINTER(Batch)
@@ -156,6 +167,13 @@ SIGNATURES = {
     "umbs_moe_route_scaled": (c_int, [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                       c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "umbs_embedding_pos": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p]),
+    "umbs_add_rows": (c_int, [c_int, c_void_p, C.POINTER(Delta), c_int, c_int, c_float, c_void_p, c_int64, c_void_p, c_void_p]),
+    "umbs_embedding_norm": (c_int, [c_int, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_int64, c_int, c_int,
+                                    c_void_p]),
+    "umbs_memory_prep": (c_int, [c_void_p, c_int64, C.POINTER(Memory), _BP, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p]),
+    "umbs_memory_run": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, C.POINTER(Memory), _BP, c_void_p, c_void_p]),
+    "umbs_gated_norm": (c_int, [c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p,
+                                c_void_p]),
     "umbs_embedding": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]),
     "umbs_embedding_scaled": (c_int, [c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p]),
 }

@@ -17,11 +17,16 @@ Every live sequence owns one slot.  A slot holds, per layer,
   * mLSTM layers: per head the matrix S with the normaliser n as one more column and the running maximum m,
     fp32 [heads, dim (vdim + 1) + 1];
   * time-mix layers: per head the matrix memory, fp32 [heads, dim, dim] (key index first), and the previous token's
-    normed activations in the token-shift state.
+    normed activations in the token-shift state;
+  * rank-one memories (gated delta rule, state-space layers): per head the matrix memory, fp32 [heads, vdim, dim] (key
+    index last), and in front of their short convolution the last taps - 1 projected rows of queries, keys and values,
+    fp32, double-buffered like the shift state;
 and on the host its position (tokens fed so far) and parity.
 A cached-attention layer with several maps per head keeps [kv_heads (maps dim + vdim)] numbers per token; one with a
 chunked mask needs a ring of one chunk only; one that borrows another layer's keys and values keeps nothing (the lender's
-ring reaches as far back as its furthest-seeing borrower reads).  A layer's second mixer (two mixers side by side) has
+ring reaches as far back as its furthest-seeing borrower reads).  A layer that runs several times (``spec.loop``) has state of
+its own for every run: the lists are indexed by layer *run* (``spec.layer_runs()``; ``state_index`` of a layer is its first
+run).  A layer's second mixer (two mixers side by side) has
 state of its own, kept behind the layers' in the same lists (``spec.layers[i].second.state_index``).  Nothing is cleared when a slot is freed or handed out
 again: the kernels read a sequence's state as zero while its position is 0, and a ring row is only ever read for a
 position that the current owner has written.
@@ -39,14 +44,21 @@ class SequenceStateCache:
         self.slots = 0
         # tokens per sequence that the growing parts (windowless key/value rows, pooled-block tables) hold
         self.capacity = int(max_length or capacity or 512)
-        # every mixer that keeps state: the layers' own, then the second mixers of layers that run two side by side
+        # every mixer that keeps state: one per layer run, then the second mixers of layers that run two side by side
         self.units = []
-        for i, l in enumerate(spec.layers):
-            l.state_index = i
-            self.units.append(l)
+        self.second_index: dict[int, int] = {}           # run -> where its second mixer's state is
+        runs = [spec.layers[i] for i, _ in spec.layer_runs()]
         for l in spec.layers:
+            l.state_index = -1
             if getattr(l, "second", None) is not None:
-                l.second.state_index = len(self.units)
+                l.second.state_index = -1
+        for r, l in enumerate(runs):
+            l.state_index = r if l.state_index < 0 else l.state_index
+            self.units.append(l)
+        for r, l in enumerate(runs):
+            if getattr(l, "second", None) is not None:
+                self.second_index[r] = len(self.units)
+                l.second.state_index = len(self.units) if l.second.state_index < 0 else l.second.state_index
                 self.units.append(l.second)
         # a layer that lends its keys and values keeps them as far back as its furthest-seeing borrower asks
         self._borrowers = {}
@@ -61,6 +73,7 @@ class SequenceStateCache:
         self.conv_state: list[torch.Tensor | None] = [None] * n
         self.mlstm_state: list[torch.Tensor | None] = [None] * n
         self.tm_state: list[torch.Tensor | None] = [None] * n
+        self.mem_state: list[torch.Tensor | None] = [None] * n
         self.shift: list[torch.Tensor | None] = [None] * n
         self.ret_state: list[torch.Tensor | None] = [None] * n
         self.ring: list[torch.Tensor | None] = [None] * n
@@ -144,6 +157,10 @@ class SequenceStateCache:
                 if l.taps > 1:
                     self.conv_state[i] = widen(self.conv_state[i], (2, slots, l.taps - 1, (l.heads + l.kv_heads) * l.maps * l.dim),
                                                1, **f32)
+            elif l.mixer in ("gated_delta", "ssd"):
+                self.mem_state[i] = widen(self.mem_state[i], (slots, l.heads, l.vdim, l.dim), 0, **f32)
+                if l.taps > 1:
+                    self.conv_state[i] = widen(self.conv_state[i], (2, slots, l.taps - 1, 2 * l.kv_heads * l.dim + l.heads * l.vdim), 1, **f32)
             elif l.mixer == "mlstm":
                 self.mlstm_state[i] = widen(self.mlstm_state[i], (slots, l.heads, l.dim * (l.vdim + 1) + 1), 0, **f32)
         self.position += [0] * (slots - old)
@@ -177,7 +194,7 @@ class SequenceStateCache:
     def state_bytes_per_slot(self) -> int:
         n = 0
         for t in self.shift + self.ret_state + self.ring + self.kv_cache + self.pool_cache + self.conv_state + self.mlstm_state + \
-                self.tm_state:
+                self.tm_state + self.mem_state:
             if t is not None:
                 n += t.numel() * t.element_size() // self.slots
         return n

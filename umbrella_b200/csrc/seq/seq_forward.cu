@@ -61,8 +61,16 @@ struct Scratch {
     void* lowrank;     // act [T, max decay_rank]
     float* wraw;       // fp32 [T, max heads dim]  the decay before its exponentials
     float* mix_out2;   // fp32 [T, width]  a second mixer's output
+    float* mem_qkv;    // fp32 [T, max channels]  a rank-one memory's convolved queries, keys and values
+    float* mem_kq;     // fp32 [T, max kv_heads]  k . q
+    void* merge;       // act [T, 2 width]  residual stream | embedding output in front of a looped pass
     std::vector<void*> kv_rows;   // per layer: the step's key | value rows (a buffer of its own for a layer others borrow from)
 };
+
+// a rank-one memory layer's channels (queries, keys, values), and their row stride in mem_qkv (16-byte rows)
+static int mem_channels(const umbs_layer_t& l) { return 2 * l.kv_heads * l.dim + l.heads * l.vdim; }
+static int mem_stride(const umbs_layer_t& l) { return (mem_channels(l) + 3) & ~3; }
+static bool is_memory(const umbs_layer_t& l) { return l.mixer == UMBS_MIX_GATED_DELTA || l.mixer == UMBS_MIX_SSD; }
 
 // layer j lends its keys and values to a later layer
 static bool lends_kv(const umbs_model_t* m, int j) {
@@ -78,7 +86,8 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
     size_t segb = 0;
     int hmax = 1, rotd = 1, in_rows = 1, hv = 1, qr = 1, kvr = 1, hd = 1, hkv = 1, hkvw = 1, top = 1, experts = 1, ff = 1, sff = 1;
     int hall = 1, cav = 1, rawd = 1, n_mix = 0, rank = 1, tmhd = 1;
-    bool parallel = false, two = false;
+    int memc = 0, memg = 0;
+    bool parallel = false, two = false, merges = false;
     auto up = [](int& a, int b) { if (b > a) a = b; };
     for (int i = 0; i < m->n_layers; ++i)
         if (m->layers[i].form == UMBS_FORM_PARALLEL) parallel = true;
@@ -87,6 +96,7 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
         if ((u & 1) && m->layers[i].second == nullptr) continue;
         const umbs_layer_t& l = (u & 1) ? *m->layers[i].second : m->layers[i];
         if (u & 1) two = true;
+        if (l.w_merge != nullptr) merges = true;
         up(hv, l.heads * l.vdim);
         up(hall, l.heads);
         if (l.mixer == UMBS_MIX_CACHED_ATTENTION) {
@@ -95,6 +105,9 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
             up(in_rows, l.heads * M * l.dim + l.kv_heads * M * l.dim + (l.values_are_keys ? 0 : l.kv_heads * l.vdim) + gate_rows);
             up(hd, l.heads * M * l.dim); up(hkvw, l.kv_heads * (M * l.dim + l.vdim)); up(cav, l.vdim);
             up(rawd, l.heads * M * (l.talk != nullptr ? l.kv_heads : 1) * l.vdim);
+        } else if (is_memory(l)) {
+            up(in_rows, mem_channels(l) + l.heads * l.vdim + (l.mixer == UMBS_MIX_SSD ? 1 : 2) * l.heads);
+            up(memc, mem_stride(l)); up(memg, l.kv_heads);
         } else if (l.mixer == UMBS_MIX_TIME_MIX) {
             up(in_rows, 4 * l.heads * l.dim); up(rank, l.decay_rank); up(tmhd, l.heads * l.dim);
             n_mix = 5;
@@ -161,6 +174,9 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
     z.lowrank = a.take(Tz * rank * es);
     z.wraw = (float*)a.take(Tz * tmhd * 4);
     z.mix_out2 = (float*)a.take(two ? Tz * W * 4 : 0);
+    z.mem_qkv = (float*)a.take(Tz * memc * 4);
+    z.mem_kq = (float*)a.take(Tz * memg * 4);
+    z.merge = a.take(merges ? Tz * 2 * W * es : 0);
     z.kv_rows.assign(m->n_layers, z.kv);
     for (int i = 0; i < m->n_layers; ++i) {
         const umbs_layer_t& l = m->layers[i];
@@ -193,8 +209,19 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
     Scratch s;
     if (carve(m, T, b->n_want, (char*)workspace, &s) > workspace_bytes) return UMB_ERR_WORKSPACE;
     const int64_t plane = (int64_t)T * W;
-    UMBS_TRY(umbs_embedding_pos(dt, b->tok_ids, b->tok_pos, m->embed, m->embed_scale != 0.f ? m->embed_scale : 1.f, m->pos_freq,
-                                s.stack, T, W, stream));
+    const float embed_scale = m->embed_scale != 0.f ? m->embed_scale : 1.f;
+    const size_t es = dt == UMBS_F32 ? 4 : 2;
+    bool merges = false;
+    for (int i = 0; i < m->n_layers; ++i) merges |= m->layers[i].w_merge != nullptr;
+    if (m->embed_norm != nullptr) {
+        // (looped passes read the embedding output again: it waits in the second half of the merge rows)
+        if (m->pos_freq != nullptr) return UMB_ERR_UNSUPPORTED;
+        UMBS_TRY(umbs_embedding_norm(dt, b->tok_ids, m->embed, embed_scale, m->embed_norm, m->norm_eps, s.stack,
+                                     merges ? (char*)s.merge + (size_t)W * es : nullptr, 2 * (int64_t)W, T, W, stream));
+    } else {
+        UMBS_TRY(umbs_embedding_pos(dt, b->tok_ids, b->tok_pos, m->embed, embed_scale, m->pos_freq, s.stack, T, W, stream));
+        if (merges) UMBS_TRY(umbs_add_rows(dt, s.stack, nullptr, T, W, 0.f, (char*)s.merge + (size_t)W * es, 2 * (int64_t)W, nullptr, stream));
+    }
     const float* x = s.stack;                    // layer 0 reads X_0 itself
     bool prenorm = false;
     for (int i = 0; i < m->n_layers; ++i) {
@@ -210,7 +237,7 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
                          void* y, float* copy) -> int {
         const bool plain = kind == UMBS_NORM_RMS && (!has_pend || (pend.pair_out == nullptr && pend.shared == nullptr &&
                                                                    pend.scale == nullptr && pend.mult == 1.f &&
-                                                                   pend.delta2 == nullptr && (pend.delta_mult == 0.f || pend.delta_mult == 1.f)));
+                                                                   pend.delta2 == nullptr && pend.norm_w == nullptr && (pend.delta_mult == 0.f || pend.delta_mult == 1.f)));
         if (plain) return umbs_add_rms_norm(dt, s.stack, has_pend ? pend.delta : nullptr, rows, n, w, off, W, m->norm_eps, y, copy, stream);
         return umbs_add_norm_ex(dt, s.stack, has_pend ? &pend : nullptr, rows, n, kind, w, bias, off, alpha, W, m->norm_eps, y, copy,
                                 stream);
@@ -255,7 +282,6 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
                 UMBS_TRY(umbs_ring_append(dt, kv_rows, l.kv_cache, l.kv_len, b, row_kv, stream));
         } else if (l.mixer == UMBS_MIX_TIME_MIX) {
             const int hd = l.heads * l.dim, rows = 4 * hd;
-            const size_t es = dt == UMBS_F32 ? 4 : 2;
             if (l.vdim != l.dim || l.mix_mu == nullptr || l.shift_state == nullptr || l.decay_rank < 1) return UMB_ERR_ARG;
             UMBS_TRY(umbs_shift_mix(dt, s.h, l.mix_mu, 5, l.shift_state, m->slots, b, W, s.mixes, stream));
             // r | k | v | g: one batched product over the first four mixes
@@ -268,6 +294,25 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
                                nullptr, nullptr, 0, 0.f, stream));
             UMBS_TRY(umbs_time_mix(dt, s.proj, rows, s.wraw, l.decay_bias, l.bonus, b, l.heads, l.dim, m->norm_eps, l.out_norm_w,
                                    l.tm_state, s.o32, s.mixed, stream));
+        } else if (is_memory(l)) {
+            // columns of the projection (see umbs_layer_t): where the gate, the convolved channels and the gates' inputs sit
+            const bool delta = l.mixer == UMBS_MIX_GATED_DELTA;
+            if (l.kv_heads < 1 || l.heads % l.kv_heads != 0 || l.mem_state == nullptr || l.out_norm_w == nullptr) return UMB_ERR_ARG;
+            const int ch = mem_channels(l), gd = l.kv_heads * l.dim, rows = ch + hv + (delta ? 2 : 1) * l.heads, ldq = mem_stride(l);
+            umbs_memory_t mem{};
+            mem.rule = delta ? UMBS_MEMORY_DELTA : UMBS_MEMORY_ADD;
+            mem.heads = l.heads; mem.kv_heads = l.kv_heads; mem.dim = l.dim; mem.vdim = l.vdim; mem.taps = l.taps;
+            mem.off_conv = delta ? 0 : hv;
+            mem.off_q = delta ? 0 : hv + gd; mem.off_k = delta ? gd : hv; mem.off_v = delta ? 2 * gd : 0;
+            mem.off_strength = delta ? ch + hv : -1; mem.off_decay = delta ? ch + hv + l.heads : hv + ch;
+            mem.unit = delta;
+            mem.conv_w = l.conv_w; mem.conv_b = l.conv_b; mem.conv_state = l.conv_state;
+            mem.decay_rate = l.decay_rate; mem.dt_bias = l.dt_bias; mem.skip = l.skip_w; mem.state = l.mem_state;
+            UMBS_TRY(umbs_gemm(dt, s.h, W, 0, l.w_in, W, 0, s.proj, rows, 0, 1, T, rows, W, 1, nullptr, nullptr, 0, 0.f, stream));
+            UMBS_TRY(umbs_memory_prep(s.proj, rows, &mem, b, m->slots, s.mem_qkv, ldq, s.gates, s.mem_kq, stream));
+            UMBS_TRY(umbs_memory_run(s.mem_qkv, ldq, s.gates, s.mem_kq, &mem, b, s.o32, stream));
+            UMBS_TRY(umbs_gated_norm(dt, s.o32, delta ? s.proj + ch : s.proj, rows, T, hv, delta ? l.heads : l.norm_parts, l.out_norm_w,
+                                     delta ? l.vdim : hv, !delta, m->norm_eps, s.mixed, stream));
         } else {
             return UMB_ERR_UNSUPPORTED;
         }
@@ -277,9 +322,17 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
         const umbs_layer_t& l = m->layers[i];
         const int hv = l.heads * l.vdim;
         const float mult = l.residual_mult != 0.f ? l.residual_mult : 1.f;
-        UMBS_TRY(norm_step(nullptr, T, l.norm_kind, l.norm_w, l.norm_b, l.norm_offset, l.norm_alpha, s.h,
-                           (layer_out && i > 0) ? layer_out + (int64_t)(i - 1) * plane : nullptr));
-        const bool generic = l.mixer == UMBS_MIX_CACHED_ATTENTION || l.mixer == UMBS_MIX_TIME_MIX;
+        float* prev_out = (layer_out && i > 0) ? layer_out + (int64_t)(i - 1) * plane : nullptr;
+        if (l.w_merge != nullptr) {
+            // a pass of a loop begins: the finished stream and the embedding output go through one product
+            UMBS_TRY(umbs_add_rows(dt, s.stack, has_pend ? &pend : nullptr, T, W, m->norm_eps, s.merge, 2 * (int64_t)W, prev_out, stream));
+            UMBS_TRY(umbs_gemm(dt, s.merge, 2 * (int64_t)W, 0, l.w_merge, 2 * (int64_t)W, 0, s.stack, W, 0, 1, T, W, 2 * W, 1, nullptr,
+                               nullptr, 0, 0.f, stream));
+            has_pend = false;
+            prev_out = nullptr;
+        }
+        UMBS_TRY(norm_step(nullptr, T, l.norm_kind, l.norm_w, l.norm_b, l.norm_offset, l.norm_alpha, s.h, prev_out));
+        const bool generic = l.mixer == UMBS_MIX_CACHED_ATTENTION || l.mixer == UMBS_MIX_TIME_MIX || is_memory(l);
         if (generic) {
             UMBS_TRY(run_mixer(l, i, s.mix_out));
             if (l.second != nullptr) UMBS_TRY(run_mixer(*l.second, i, s.mix_out2));
@@ -312,7 +365,6 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
                 // a step of fresh sequences: every visible key is in the step, so every head's own key part and its values
                 // are up-projected once per token and a (row, key) pair costs dim + rope_dim + vdim multiply-adds
                 const int hdk = l.heads * l.dim;
-                const size_t es = dt == UMBS_F32 ? 4 : 2;
                 UMBS_TRY(umbs_gemm(dt, s.c, KD, 0, l.w_ukv, R, 0, s.kv, hdk + hv, 0, 0, T, hdk + hv, R, 1, nullptr, nullptr, 0, 0.f,
                                    stream));
                 UMBS_TRY(umbs_window_attention_ex(dt, s.q, hdq, s.kv, hdk + hv, (const char*)s.c + (size_t)R * es, KD, Rt,
@@ -341,6 +393,7 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
         pend = umbs_delta_t{};
         pend.delta = s.mix_out; pend.scale = l.out_scale; pend.mult = mult;
         pend.delta_mult = 1.f;
+        pend.norm_w = l.post_norm_w;
         if (l.second != nullptr) {           // two mixers side by side: both factors as given (0 is a factor like any other)
             pend.delta_mult = l.mix_scale;
             pend.delta2 = s.mix_out2; pend.delta2_mult = l.second_scale;
@@ -352,7 +405,7 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
             const int act = f.act ? f.act : UMBS_ACT_CLAMPED_GLU;
             UMBS_TRY(norm_step(nullptr, T, l.norm_kind, l.norm2_w, l.norm2_b, l.norm_offset, l.norm2_alpha, s.h, nullptr));
             pend = umbs_delta_t{};
-            pend.scale = l.out_scale2; pend.mult = mult;
+            pend.scale = l.out_scale2; pend.mult = mult; pend.norm_w = l.post_norm2_w;
             if (f.experts > 0) {
                 // (the shared expert's per-token gate rides along as one more row of the router)
                 UMBS_TRY(umbs_moe_route_scaled(dt, s.h, T, W, f.w_router, f.experts, f.top, f.route_mode, f.groups, f.keep,
@@ -397,6 +450,7 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
         }
         return 0;
     }
+    if (merges) return UMB_ERR_UNSUPPORTED;
     for (int i = 0; i < m->n_layers; ++i) {
         const umbs_layer_t& l = m->layers[i];
         UMBS_TRY(umbs_group_norm_shift(dt, x, l.norm_w, l.shift_w, l.shift_state, m->slots, b, W, m->norm_groups,

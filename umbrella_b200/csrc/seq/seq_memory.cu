@@ -1,0 +1,398 @@
+// Rank-one memories: matrix states with one decay and one write strength per head and token -- the gated delta rule and
+// state-space layers (see umbs_memory_t in include/umbrella_b200_seq.h).  fp32 arithmetic throughout; the state is fp32
+// [slots, heads, vdim, dim], key index last, so that a value column is contiguous.
+//
+//   umbs_memory_prep : short causal convolution + silu, unit norms of q and k, decay and strength, the dot product k . q.
+//   umbs_memory_run  : the recurrence, one block per (value columns, head, sequence).
+//   umbs_gated_norm  : unit RMS of the parts of the output, weight, silu gate (in front of the norm or behind it).
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <math.h>
+#include <stdint.h>
+
+#include "seq_internal.h"
+
+namespace umbs {
+
+__device__ __forceinline__ float warp_sum_mem(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ float silu_mem(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float softplus_mem(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+// ------------------------------------------------------------------------------------------------ preparation
+constexpr int kPrepWarps = 4, kPrepVals = 4;       // warps per block; channels per lane of a value task
+
+// A warp's task: one query / key head (both vectors, their norms and their dot product), 128 value channels, or the gates
+// of all heads -- for `tile` consecutive tokens, so that the rows a convolution shares with its neighbours are read through
+// L1.  A lane's sums run in a fixed order, so a token's result does not depend on what else is in the step.
+template <int NC>
+__global__ void __launch_bounds__(32 * kPrepWarps) memory_prep_kernel(const float* __restrict__ proj, int64_t ld, umbs_memory_t m, Batch b,
+                                                                      int slots, int tile, float* __restrict__ qkv, int64_t ld_qkv,
+                                                                      float* __restrict__ gates, float* __restrict__ kq) {
+    const int lane = threadIdx.x & 31, task = blockIdx.y * kPrepWarps + (threadIdx.x >> 5);
+    const int G = m.kv_heads, D = m.dim, cv = m.heads * m.vdim, C = 2 * G * D + cv, taps = m.taps, keep = taps - 1;
+    const int vtasks = (cv + 32 * kPrepVals - 1) / (32 * kPrepVals);
+    if (task > G + vtasks) return;
+    const int t_end = min(b.n_tokens, (int)(blockIdx.x + 1) * tile);
+    for (int t = blockIdx.x * tile; t < t_end; ++t) {
+        if (task == G + vtasks) {
+            const float* row = proj + (int64_t)t * ld;
+            for (int h = lane; h < m.heads; h += 32) {
+                const float dt = softplus_mem(row[m.off_decay + h] + m.dt_bias[h]);
+                float* g = gates + ((int64_t)t * m.heads + h) * 2;
+                g[0] = -m.decay_rate[h] * dt;
+                g[1] = m.off_strength >= 0 ? 1.f / (1.f + expf(-row[m.off_strength + h])) : dt;
+            }
+            continue;
+        }
+        const int s = b.tok_seq[t], pos = b.tok_pos[t];
+        const int start = b.seq_start[s], len = b.seq_len[s], pos0 = b.seq_pos0[s], slot = b.seq_slot[s], par = b.seq_parity[s];
+        const float* st_in = keep > 0 ? m.conv_state + ((int64_t)par * slots + slot) * keep * C : nullptr;
+        // the projected value of channel c at position p: this step's row, the carried rows, or zero in front of the sequence
+        auto u_at = [&](int c, int p) -> float {
+            if (p >= pos0) return proj[(int64_t)(start + p - pos0) * ld + m.off_conv + c];
+            return p < 0 ? 0.f : st_in[(int64_t)(p - (pos0 - keep)) * C + c];
+        };
+        auto conv = [&](int c) -> float {
+            float acc = m.conv_b != nullptr ? m.conv_b[c] : 0.f;
+            for (int j = 0; j < taps; ++j) acc = fmaf(m.conv_w[(int64_t)c * taps + j], u_at(c, pos - keep + j), acc);
+            return silu_mem(acc);
+        };
+        // the sequence's last token of the step leaves the rows the next step starts from (the other half of the buffer)
+        const bool last = keep > 0 && t == start + len - 1;
+        float* st_out = last ? m.conv_state + ((int64_t)(par ^ 1) * slots + slot) * keep * C : nullptr;
+        auto carry = [&](int c) {
+            for (int r = 0; r < keep; ++r) st_out[(int64_t)r * C + c] = u_at(c, pos0 + len - keep + r);
+        };
+        float* out = qkv + (int64_t)t * ld_qkv;
+        if (task < G) {
+            const int cq = m.off_q + task * D, ck = m.off_k + task * D;
+            float q[NC], k[NC], qq = 0.f, kk = 0.f, dot = 0.f;
+#pragma unroll
+            for (int i = 0; i < NC; ++i) {
+                const int d = lane + 32 * i;
+                q[i] = k[i] = 0.f;
+                if (d < D) {
+                    q[i] = conv(cq + d);
+                    k[i] = conv(ck + d);
+                    qq = fmaf(q[i], q[i], qq);
+                    kk = fmaf(k[i], k[i], kk);
+                    if (last) { carry(cq + d); carry(ck + d); }
+                }
+            }
+            float fq = 1.f, fk = 1.f;
+            if (m.unit) {
+                fq = 1.f / sqrtf(warp_sum_mem(qq) + 1e-6f) * (1.f / sqrtf((float)D));
+                fk = 1.f / sqrtf(warp_sum_mem(kk) + 1e-6f);
+            }
+#pragma unroll
+            for (int i = 0; i < NC; ++i) {
+                const int d = lane + 32 * i;
+                q[i] *= fq;
+                k[i] *= fk;
+                dot = fmaf(q[i], k[i], dot);
+                if (d < D) { out[cq + d] = q[i]; out[ck + d] = k[i]; }
+            }
+            dot = warp_sum_mem(dot);
+            if (lane == 0) kq[(int64_t)t * G + task] = dot;
+        } else {
+            const int c0 = (task - G) * 32 * kPrepVals;
+#pragma unroll
+            for (int i = 0; i < kPrepVals; ++i) {
+                const int c = c0 + lane + 32 * i;
+                if (c >= cv) continue;
+                out[m.off_v + c] = conv(m.off_v + c);
+                if (last) carry(m.off_v + c);
+            }
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ recurrence
+constexpr int kMemWarps = 4, kMemStages = 3;
+
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src));
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src));
+}
+
+// RL lanes share a value column and hold RPL of its rows each (rows 4 (r + RL i) .. + 3 of lane r, so that the 16-byte loads
+// of the lanes that share a column are consecutive); a lane holds CPL columns.  The whole state slice stays in registers for
+// the step.  Tokens run in order; TB at a time are staged (q, k, the block's value columns, decay, strength, k . q) in a ring
+// of shared-memory stages filled by asynchronous copies.  Both products with the state use the state in front of the
+// token's write, S^T q after it being decay (S^T q) + (k . q) u, so one pass over the rows and one round of shuffles serve
+// the write and the read-out.  The order of every addition is fixed by the layout: a token's result does not depend on how
+// the sequence was cut into steps.
+template <int RL, int RPL, int CPL, int TB, bool DELTA>
+__global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __restrict__ qkv, int64_t ld, const float* __restrict__ gates,
+                                                                const float* __restrict__ kq, umbs_memory_t m, Batch b,
+                                                                float* __restrict__ o, int vec) {
+    constexpr int DP = RL * RPL, WC = 32 / RL * CPL, CT = kMemWarps * WC;         // padded rows; columns per warp and per block
+    constexpr int STAGE = TB * (2 * DP + CT + 4);
+    extern __shared__ __align__(16) float mem_sm[];
+    float* so = mem_sm + kMemStages * STAGE;                                       // [TB][CT]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rl = lane % RL, cl = lane / RL;
+    const int h = blockIdx.y, s = blockIdx.z, c0 = blockIdx.x * CT, D = m.dim, V = m.vdim;
+    const int grp = h / (m.heads / m.kv_heads);
+    const int start = b.seq_start[s], len = b.seq_len[s], pos0 = b.seq_pos0[s], slot = b.seq_slot[s];
+    const int cq = m.off_q + grp * D, ck = m.off_k + grp * D, cv = m.off_v + h * V + c0;
+    const int hv = m.heads * V, ncol = min(CT, V - c0);
+    const float skip = m.skip != nullptr ? m.skip[h] : 0.f;
+    float* st = m.state + ((int64_t)slot * m.heads + h) * V * D;                   // S[column][row]
+    float S[CPL][RPL];
+    int col[CPL];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+        col[c] = warp * WC + c * (32 / RL) + cl;
+        const float* sc = st + (int64_t)(c0 + col[c]) * D;
+        const bool have = pos0 > 0 && col[c] < ncol;
+#pragma unroll
+        for (int i = 0; i < RPL / 4; ++i) {
+            const int r = 4 * (rl + RL * i);
+            if (have && D % 4 == 0) {
+                const float4 f = r < D ? *reinterpret_cast<const float4*>(sc + r) : make_float4(0.f, 0.f, 0.f, 0.f);
+                S[c][4 * i] = f.x; S[c][4 * i + 1] = f.y; S[c][4 * i + 2] = f.z; S[c][4 * i + 3] = f.w;
+            } else {
+#pragma unroll
+                for (int x = 0; x < 4; ++x) S[c][4 * i + x] = (have && r + x < D) ? sc[r + x] : 0.f;
+            }
+        }
+    }
+    // rows beyond dim and columns beyond vdim of every stage stay zero
+    for (int i = tid; i < kMemStages * STAGE; i += 32 * kMemWarps) mem_sm[i] = 0.f;
+    __syncthreads();
+    auto issue = [&](int g) {
+        float* sq = mem_sm + (g % kMemStages) * STAGE;
+        float* sk = sq + TB * DP;
+        float* sv = sk + TB * DP;
+        float* sg = sv + TB * CT;                                                  // [3][TB] decay, strength, k . q
+        const int t0 = g * TB, nt = min(TB, len - t0);
+        const float* base = qkv + (int64_t)(start + t0) * ld;
+        if (vec) {
+            const int p = D / 4;
+            for (int i = tid; i < nt * p; i += 32 * kMemWarps) {
+                const int tt = i / p, d = (i - tt * p) * 4;
+                cp_async16(sq + tt * DP + d, base + (int64_t)tt * ld + cq + d);
+                cp_async16(sk + tt * DP + d, base + (int64_t)tt * ld + ck + d);
+            }
+            for (int i = tid; i < nt * (CT / 4); i += 32 * kMemWarps) {
+                const int tt = i / (CT / 4), d = (i - tt * (CT / 4)) * 4;
+                if (d < ncol) cp_async16(sv + tt * CT + d, base + (int64_t)tt * ld + cv + d);
+            }
+        } else {
+            for (int i = tid; i < nt * D; i += 32 * kMemWarps) {
+                const int tt = i / D, d = i - tt * D;
+                cp_async4(sq + tt * DP + d, base + (int64_t)tt * ld + cq + d);
+                cp_async4(sk + tt * DP + d, base + (int64_t)tt * ld + ck + d);
+            }
+            for (int i = tid; i < nt * CT; i += 32 * kMemWarps) {
+                const int tt = i / CT, d = i - tt * CT;
+                if (d < ncol) cp_async4(sv + tt * CT + d, base + (int64_t)tt * ld + cv + d);
+            }
+        }
+        if (tid < nt) {
+            const int64_t t = start + t0 + tid;
+            cp_async4(sg + tid, gates + (t * m.heads + h) * 2);
+            cp_async4(sg + TB + tid, gates + (t * m.heads + h) * 2 + 1);
+            cp_async4(sg + 2 * TB + tid, kq + t * m.kv_heads + grp);
+        }
+    };
+    const int groups = (len + TB - 1) / TB;
+    for (int g = 0; g < kMemStages - 1; ++g) {
+        if (g < groups) issue(g);
+        asm volatile("cp.async.commit_group;\n" ::);
+    }
+    for (int g = 0; g < groups; ++g) {
+        // (the stage this writes was walked in the previous iteration, which ended with a barrier)
+        if (g + kMemStages - 1 < groups) issue(g + kMemStages - 1);
+        asm volatile("cp.async.commit_group;\n" ::);
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(kMemStages - 1));           // this thread's copies of group g have landed
+        float* sq = mem_sm + (g % kMemStages) * STAGE;
+        float* sk = sq + TB * DP;
+        float* sv = sk + TB * DP;
+        float* sg = sv + TB * CT;
+        const int t0 = g * TB, nt = min(TB, len - t0);
+        if (tid < nt) sg[tid] = expf(sg[tid]);                                     // (the thread that copied it)
+        __syncthreads();
+        for (int tt = 0; tt < nt; ++tt) {
+            const float dec = sg[tt], str = sg[TB + tt], dot = sg[2 * TB + tt];
+            float k[RPL], aq[CPL][4], ak[CPL][4];
+#pragma unroll
+            for (int c = 0; c < CPL; ++c)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) aq[c][x] = ak[c][x] = 0.f;
+#pragma unroll
+            for (int i = 0; i < RPL / 4; ++i) {
+                const float4 k4 = *reinterpret_cast<const float4*>(sk + tt * DP + 4 * (rl + RL * i));
+                const float4 q4 = *reinterpret_cast<const float4*>(sq + tt * DP + 4 * (rl + RL * i));
+                k[4 * i] = k4.x; k[4 * i + 1] = k4.y; k[4 * i + 2] = k4.z; k[4 * i + 3] = k4.w;
+                const float qa[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+                for (int c = 0; c < CPL; ++c)
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) {
+                        if (DELTA) ak[c][x] = fmaf(S[c][4 * i + x], k[4 * i + x], ak[c][x]);
+                        aq[c][x] = fmaf(S[c][4 * i + x], qa[x], aq[c][x]);
+                    }
+            }
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) {
+                float dq = (aq[c][0] + aq[c][1]) + (aq[c][2] + aq[c][3]);
+                float dk = (ak[c][0] + ak[c][1]) + (ak[c][2] + ak[c][3]);
+#pragma unroll
+                for (int w = RL / 2; w > 0; w >>= 1) {
+                    if (DELTA) dk += __shfl_xor_sync(0xffffffffu, dk, w);
+                    dq += __shfl_xor_sync(0xffffffffu, dq, w);
+                }
+                const float v = sv[tt * CT + col[c]];
+                const float u = DELTA ? str * fmaf(-dec, dk, v) : str * v;
+#pragma unroll
+                for (int i = 0; i < RPL; ++i) S[c][i] = fmaf(dec, S[c][i], k[i] * u);
+                if (rl == 0) so[tt * CT + col[c]] = fmaf(skip, v, fmaf(dot, u, dec * dq));
+            }
+        }
+        __syncthreads();
+        for (int i = tid; i < nt * CT; i += 32 * kMemWarps) {
+            const int tt = i / CT, c = i - tt * CT;
+            if (c < ncol) o[(int64_t)(start + t0 + tt) * hv + h * V + c0 + c] = so[i];
+        }
+    }
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+        if (col[c] >= ncol) continue;
+        float* sc = st + (int64_t)(c0 + col[c]) * D;
+#pragma unroll
+        for (int i = 0; i < RPL / 4; ++i) {
+            const int r = 4 * (rl + RL * i);
+            if (D % 4 == 0) {
+                if (r < D) *reinterpret_cast<float4*>(sc + r) = make_float4(S[c][4 * i], S[c][4 * i + 1], S[c][4 * i + 2], S[c][4 * i + 3]);
+            } else {
+#pragma unroll
+                for (int x = 0; x < 4; ++x)
+                    if (r + x < D) sc[r + x] = S[c][4 * i + x];
+            }
+        }
+    }
+}
+
+template <int RL, int RPL, int CPL, int TB, bool DELTA>
+static int launch_memory(const float* qkv, int64_t ld, const float* gates, const float* kq, const umbs_memory_t& m, const Batch& b, float* o,
+                         int vec, cudaStream_t st) {
+    constexpr int CT = kMemWarps * (32 / RL * CPL);
+    constexpr size_t smem = ((size_t)kMemStages * TB * (2 * RL * RPL + CT + 4) + (size_t)TB * CT) * sizeof(float);
+    static bool set = false;
+    if (smem > 48 * 1024 && !set) {
+        cudaError_t e = cudaFuncSetAttribute(memory_kernel<RL, RPL, CPL, TB, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+        set = true;
+    }
+    const dim3 grid((m.vdim + CT - 1) / CT, m.heads, b.n_seqs);
+    memory_kernel<RL, RPL, CPL, TB, DELTA><<<grid, 32 * kMemWarps, smem, st>>>(qkv, ld, gates, kq, m, b, o, vec);
+    return 0;
+}
+
+// ------------------------------------------------------------------------------------------------ gated norm
+// A warp (or, for long parts, a block) per part of a row.
+template <typename T>
+__global__ void gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int64_t ldg, int n_parts, int width, int parts,
+                                  const float* __restrict__ w, int w_len, int gate_first, float eps, int whole_block, T* __restrict__ out) {
+    __shared__ float red[32];
+    const int nw = blockDim.x >> 5, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int p = whole_block ? blockIdx.x : blockIdx.x * nw + warp;
+    const int me = whole_block ? threadIdx.x : lane, step = whole_block ? blockDim.x : 32;
+    if (p >= n_parts) return;                       // (never a part of a block that meets the barrier below)
+    const int t = p / parts, size = width / parts, e0 = (p - t * parts) * size;
+    const float* orow = o + (int64_t)t * width + e0;
+    const float* grow = gate + (int64_t)t * ldg + e0;
+    float ss = 0.f;
+    for (int e = me; e < size; e += step) {
+        const float y = gate_first ? orow[e] * silu_mem(grow[e]) : orow[e];
+        ss = fmaf(y, y, ss);
+    }
+    ss = warp_sum_mem(ss);
+    if (whole_block) {
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        ss = warp_sum_mem(lane < nw ? red[lane] : 0.f);
+    }
+    const float inv = 1.f / sqrtf(ss / (float)size + eps);
+    for (int e = me; e < size; e += step)
+        out[(int64_t)t * width + e0 + e] = from_f32<T>(orow[e] * silu_mem(grow[e]) * inv * w[(e0 + e) % w_len]);
+}
+
+}  // namespace umbs
+
+using namespace umbs;
+
+static int check_memory(const umbs_memory_t* m) {
+    if (m == nullptr || m->heads < 1 || m->kv_heads < 1 || m->heads % m->kv_heads != 0 || m->dim < 1 || m->vdim < 1) return UMB_ERR_ARG;
+    if (m->rule != UMBS_MEMORY_ADD && m->rule != UMBS_MEMORY_DELTA) return UMB_ERR_ARG;
+    return m->dim > 512 ? UMB_ERR_UNSUPPORTED : 0;
+}
+
+extern "C" int umbs_memory_prep(const float* proj, int64_t ld, const umbs_memory_t* m, const umbs_batch_t* batch, int slots, float* qkv,
+                                int64_t ld_qkv, float* gates, float* kq, umbs_stream_t stream) {
+    if (batch->n_tokens <= 0) return 0;
+    const int rc = check_memory(m);
+    if (rc) return rc;
+    if (proj == nullptr || qkv == nullptr || gates == nullptr || kq == nullptr || m->taps < 1 || m->conv_w == nullptr ||
+        m->decay_rate == nullptr || m->dt_bias == nullptr || (m->taps > 1 && m->conv_state == nullptr))
+        return UMB_ERR_ARG;
+    cudaStream_t st = (cudaStream_t)stream;
+    const int tasks = m->kv_heads + (m->heads * m->vdim + 32 * kPrepVals - 1) / (32 * kPrepVals) + 1;
+    const int tile = batch->n_tokens > 256 ? 8 : 1;
+    const dim3 grid((batch->n_tokens + tile - 1) / tile, (tasks + kPrepWarps - 1) / kPrepWarps);
+    if (m->dim <= 64) memory_prep_kernel<2><<<grid, 32 * kPrepWarps, 0, st>>>(proj, ld, *m, *batch, slots, tile, qkv, ld_qkv, gates, kq);
+    else if (m->dim <= 128) memory_prep_kernel<4><<<grid, 32 * kPrepWarps, 0, st>>>(proj, ld, *m, *batch, slots, tile, qkv, ld_qkv, gates, kq);
+    else memory_prep_kernel<16><<<grid, 32 * kPrepWarps, 0, st>>>(proj, ld, *m, *batch, slots, tile, qkv, ld_qkv, gates, kq);
+    count_launches(1);
+    return (int)cudaGetLastError();
+}
+
+extern "C" int umbs_memory_run(const float* qkv, int64_t ld_qkv, const float* gates, const float* kq, const umbs_memory_t* m,
+                               const umbs_batch_t* batch, float* o, umbs_stream_t stream) {
+    if (batch->n_tokens <= 0) return 0;
+    const int rc0 = check_memory(m);
+    if (rc0) return rc0;
+    if (qkv == nullptr || gates == nullptr || kq == nullptr || o == nullptr || m->state == nullptr) return UMB_ERR_ARG;
+    cudaStream_t st = (cudaStream_t)stream;
+    // 16-byte copies: every row, head and column tile must start on a 16-byte boundary
+    const int vec = m->dim % 4 == 0 && m->vdim % 4 == 0 && ld_qkv % 4 == 0 && m->off_q % 4 == 0 && m->off_k % 4 == 0 && m->off_v % 4 == 0 &&
+                    (uintptr_t)qkv % 16 == 0;
+#define UMBS_MEM(RL, RPL, TB)                                                                                                     \
+    (m->rule == UMBS_MEMORY_DELTA ? launch_memory<RL, RPL, 1, TB, true>(qkv, ld_qkv, gates, kq, *m, *batch, o, vec, st)            \
+                                  : launch_memory<RL, RPL, 1, TB, false>(qkv, ld_qkv, gates, kq, *m, *batch, o, vec, st))
+    int rc;
+    if (m->dim <= 32) rc = UMBS_MEM(8, 4, 16);
+    else if (m->dim <= 64) rc = UMBS_MEM(8, 8, 16);
+    else if (m->dim <= 128) rc = UMBS_MEM(8, 16, 16);
+    else if (m->dim <= 256) rc = UMBS_MEM(8, 32, 8);
+    else rc = UMBS_MEM(16, 32, 8);
+#undef UMBS_MEM
+    if (rc) return rc;
+    count_launches(1);
+    return (int)cudaGetLastError();
+}
+
+extern "C" int umbs_gated_norm(int dtype, const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w,
+                               int w_len, int gate_first, float eps, void* out, umbs_stream_t stream) {
+    if (n <= 0) return 0;
+    if (o == nullptr || gate == nullptr || w == nullptr || out == nullptr || parts < 1 || width % parts != 0 || w_len < 1) return UMB_ERR_ARG;
+    cudaStream_t st = (cudaStream_t)stream;
+    const int size = width / parts, n_parts = n * parts, block = size > 256;
+    const int threads = block ? (size >= 2048 ? 512 : 256) : 128;
+    const unsigned grid = block ? n_parts : (n_parts + 3) / 4;
+    if (dtype == UMBS_BF16)
+        gated_norm_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block,
+                                                                   (__nv_bfloat16*)out);
+    else if (dtype == UMBS_F32)
+        gated_norm_kernel<float><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, (float*)out);
+    else return UMB_ERR_ARG;
+    count_launches(1);
+    return (int)cudaGetLastError();
+}

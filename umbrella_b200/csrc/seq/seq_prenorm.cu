@@ -94,10 +94,12 @@ __device__ __forceinline__ float block_sum_pn(float v, float* red) {
     return red[32];
 }
 
+constexpr int kNormNone = -1;          // y gets the row as it is (umbs_add_rows)
+
 template <typename T>
 __global__ void add_norm_kernel(float* __restrict__ x, umbs_delta_t d, int has_d, const int32_t* __restrict__ rows, int kind,
                                 const float* __restrict__ w, const float* __restrict__ bias, float w_offset, float alpha, int width,
-                                float eps, T* __restrict__ y, float* __restrict__ copy) {
+                                float eps, T* __restrict__ y, int64_t ldy, float* __restrict__ copy) {
     __shared__ float red[33];
     constexpr int KEEP = 8, TOPS = 16;              // up to TOPS routed pairs per token are held in shared memory
     __shared__ float s_w[TOPS];
@@ -127,18 +129,30 @@ __global__ void add_norm_kernel(float* __restrict__ x, umbs_delta_t d, int has_d
             if (e < width) ff[i] = fmaf(wk, pk[e], ff[i]);
         }
     }
-    float sum = 0.f;
+    float sum = 0.f, dsum = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int e = threadIdx.x + i * blockDim.x;
+        float dl = 0.f;
+        if (e < width && has_d) {
+            if (d.delta != nullptr) dl = d.delta[src * width + e] * d.delta_mult;
+            if (d.delta2 != nullptr) dl = fmaf(d.delta2[src * width + e], d.delta2_mult, dl);
+            dl += ff[i];
+            if (d.shared != nullptr) dl = fmaf(d.shared[src * width + e], sg, dl);
+        }
+        ff[i] = dl;                                       // the block's whole output
+        dsum = fmaf(dl, dl, dsum);
+    }
+    const bool post = has_d && d.norm_w != nullptr;       // a norm behind the block: its output's own statistics first
+    const float dinv = post ? 1.f / sqrtf(block_sum_pn(dsum, red) / (float)width + eps) : 1.f;
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
         const int e = threadIdx.x + i * blockDim.x;
         v[i] = 0.f;
         if (e < width) {
-            float dl = 0.f;
+            float dl = ff[i];
+            if (post) dl = dl * dinv * d.norm_w[e];
             if (has_d) {
-                if (d.delta != nullptr) dl = d.delta[src * width + e] * d.delta_mult;
-                if (d.delta2 != nullptr) dl = fmaf(d.delta2[src * width + e], d.delta2_mult, dl);
-                dl += ff[i];
-                if (d.shared != nullptr) dl = fmaf(d.shared[src * width + e], sg, dl);
                 if (d.scale != nullptr) dl *= d.scale[e];
                 dl *= d.mult;
             }
@@ -147,7 +161,7 @@ __global__ void add_norm_kernel(float* __restrict__ x, umbs_delta_t d, int has_d
         }
     }
     float mean = 0.f, inv = 0.f;
-    if (y != nullptr && kind != UMBS_NORM_DYT) {          // (the tanh norm takes no statistics)
+    if (y != nullptr && kind != UMBS_NORM_DYT && kind != kNormNone) {          // (the tanh norm takes no statistics)
         sum = block_sum_pn(sum, red);
         if (kind == UMBS_NORM_LAYER) {
             mean = sum / (float)width;
@@ -167,11 +181,34 @@ __global__ void add_norm_kernel(float* __restrict__ x, umbs_delta_t d, int has_d
             if (write_x) xr[e] = v[i];
             if (copy != nullptr) copy[(int64_t)r * width + e] = v[i];
             if (y != nullptr) {
-                float o = kind == UMBS_NORM_DYT ? tanhf(alpha * v[i]) * (w_offset + w[e]) : (v[i] - mean) * inv * (w_offset + w[e]);
-                if (kind != UMBS_NORM_RMS && bias != nullptr) o += bias[e];
-                y[(int64_t)r * width + e] = from_f32<T>(o);
+                float o = v[i];
+                if (kind != kNormNone) {
+                    o = kind == UMBS_NORM_DYT ? tanhf(alpha * v[i]) * (w_offset + w[e]) : (v[i] - mean) * inv * (w_offset + w[e]);
+                    if (kind != UMBS_NORM_RMS && bias != nullptr) o += bias[e];
+                }
+                y[(int64_t)r * ldy + e] = from_f32<T>(o);
             }
         }
+    }
+}
+
+// One block per token: the embedding row through an RMS norm, in fp32 and (for a product that reads it) as T.
+template <typename T>
+__global__ void embedding_norm_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float scale, const float* __restrict__ w,
+                                      float eps, float* __restrict__ y, T* __restrict__ y2, int64_t ld2, int width) {
+    __shared__ float red[33];
+    const int t = blockIdx.x;
+    const T* row = table + (int64_t)ids[t] * width;
+    float ss = 0.f;
+    for (int e = threadIdx.x; e < width; e += blockDim.x) {
+        const float v = to_f32(row[e]) * scale;
+        ss = fmaf(v, v, ss);
+    }
+    const float inv = 1.f / sqrtf(block_sum_pn(ss, red) / (float)width + eps);
+    for (int e = threadIdx.x; e < width; e += blockDim.x) {
+        const float v = to_f32(row[e]) * scale * inv * w[e];
+        y[(int64_t)t * width + e] = v;
+        if (y2 != nullptr) y2[(int64_t)t * ld2 + e] = from_f32<T>(v);
     }
 }
 
@@ -362,12 +399,9 @@ extern "C" int umbs_add_norm(int dtype, float* x, const umbs_delta_t* d, const i
     return umbs_add_norm_ex(dtype, x, d, rows, n, kind, w, b, w_offset, 1.f, width, eps, y, copy, stream);
 }
 
-extern "C" int umbs_add_norm_ex(int dtype, float* x, const umbs_delta_t* d, const int32_t* rows, int n, int kind, const float* w,
-                                const float* b, float w_offset, float alpha, int width, float eps, void* y, float* copy,
-                                umbs_stream_t stream) {
-    if (n <= 0) return 0;
-    if (x == nullptr || width <= 0 || (y != nullptr && w == nullptr)) return UMB_ERR_ARG;
-    if (kind != UMBS_NORM_RMS && kind != UMBS_NORM_LAYER && kind != UMBS_NORM_DYT) return UMB_ERR_ARG;
+static int add_norm_run(int dtype, float* x, const umbs_delta_t* d, const int32_t* rows, int n, int kind, const float* w,
+                        const float* b, float w_offset, float alpha, int width, float eps, void* y, int64_t ldy, float* copy,
+                        umbs_stream_t stream) {
     if (width > 8192) return UMB_ERR_UNSUPPORTED;                 // a row lives in the block's registers
     if (d != nullptr && d->pair_out != nullptr && (d->sel_w == nullptr || d->pair_pos == nullptr || d->top < 1)) return UMB_ERR_ARG;
     cudaStream_t st = (cudaStream_t)stream;
@@ -377,7 +411,34 @@ extern "C" int umbs_add_norm_ex(int dtype, float* x, const umbs_delta_t* d, cons
     if (d != nullptr) dd = *d;
     if (dd.delta_mult == 0.f && dd.delta2 == nullptr) dd.delta_mult = 1.f;
     UMBS_DISPATCH_T(dtype, add_norm_kernel<T><<<n, threads, 0, st>>>(x, dd, d != nullptr, rows, kind, w, b, w_offset, alpha, width,
-                                                                     eps, (T*)y, copy));
+                                                                     eps, (T*)y, ldy, copy));
+    count_launches(1);
+    return (int)cudaGetLastError();
+}
+
+extern "C" int umbs_add_norm_ex(int dtype, float* x, const umbs_delta_t* d, const int32_t* rows, int n, int kind, const float* w,
+                                const float* b, float w_offset, float alpha, int width, float eps, void* y, float* copy,
+                                umbs_stream_t stream) {
+    if (n <= 0) return 0;
+    if (x == nullptr || width <= 0 || (y != nullptr && w == nullptr)) return UMB_ERR_ARG;
+    if (kind != UMBS_NORM_RMS && kind != UMBS_NORM_LAYER && kind != UMBS_NORM_DYT) return UMB_ERR_ARG;
+    return add_norm_run(dtype, x, d, rows, n, kind, w, b, w_offset, alpha, width, eps, y, width, copy, stream);
+}
+
+extern "C" int umbs_add_rows(int dtype, float* x, const umbs_delta_t* d, int n, int width, float eps, void* y, int64_t ldy, float* copy,
+                             umbs_stream_t stream) {
+    if (n <= 0) return 0;
+    if (x == nullptr || width <= 0 || y == nullptr || ldy < width) return UMB_ERR_ARG;
+    return add_norm_run(dtype, x, d, nullptr, n, kNormNone, nullptr, nullptr, 0.f, 1.f, width, eps, y, ldy, copy, stream);
+}
+
+extern "C" int umbs_embedding_norm(int dtype, const int32_t* ids, const void* table, float scale, const float* w, float eps, float* y,
+                                   void* y2, int64_t ld2, int n, int width, umbs_stream_t stream) {
+    if (n <= 0) return 0;
+    if (ids == nullptr || table == nullptr || w == nullptr || y == nullptr || width <= 0) return UMB_ERR_ARG;
+    const int threads = width >= 1024 ? 256 : (width >= 256 ? 128 : 64);
+    UMBS_DISPATCH_T(dtype, embedding_norm_kernel<T><<<n, threads, 0, (cudaStream_t)stream>>>(ids, (const T*)table, scale, w, eps, y, (T*)y2,
+                                                                                           ld2, width));
     count_launches(1);
     return (int)cudaGetLastError();
 }

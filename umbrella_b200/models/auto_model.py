@@ -64,8 +64,14 @@ def _subivik(path, **kw):
     return subivik.from_pretrained(path, **kw)
 
 
+def _ralapel(path, **kw):
+    from . import ralapel
+    return ralapel.from_pretrained(path, **kw)
+
+
 # config.json ``architecture`` -> factory(path, device=, dtype=, max_length=, slots=, max_tokens=, ...)
-_ARCHITECTURES = {"Radanex": _radanex, "Zedotar": _zedotar, "Kulisun": _kulisun, "Subivik": _subivik}
+_ARCHITECTURES = {"Radanex": _radanex, "Zedotar": _zedotar, "Kulisun": _kulisun, "Subivik": _subivik,
+                  "Ralapel": _ralapel}
 
 
 def _make(model_name, offload=False, batch_size=1, max_length=None, device="cuda:0", dtype=torch.float16, **unused):

@@ -4,10 +4,11 @@ A model is a ``SeqModelSpec``: width, vocabulary, the norm's constants and a lis
 its form (``"parallel"``: one grouped norm feeds mixer and feed-forward side by side, with token shift and a depth
 average as options; ``"prenorm"``: x += mixer(norm1(x)), x += ff(norm2(x)), RMS or layer norms, optionally with a learned
 scale vector and a multiplier on every block's output), its mixer (``"retention"``, ``"latent_attention"``,
-``"cached_attention"``, ``"mlstm"`` or ``"time_mix"``) with that mixer's sizes and constants -- a pre-norm layer may run a
+``"cached_attention"``, ``"mlstm"``, ``"time_mix"``, ``"gated_delta"`` or ``"ssd"``) with that mixer's sizes and constants -- a pre-norm layer may run a
 second mixer beside the first (``second``), both reading the same normed rows --, and its feed-forward (routed experts and /
-or a shared expert -- a dense feed-forward is a shared expert alone -- or none).  Model families (models/radanex.py,
-models/zedotar.py, models/kulisun.py) translate their config.json into a spec and their tensors into the per-layer
+or a shared expert -- a dense feed-forward is a shared expert alone -- or none).  A span of layers may run several times in a
+row with the same weights (``loop``), every run with state of its own.  Model families (models/radanex.py, models/zedotar.py,
+models/kulisun.py, models/subivik.py, models/ralapel.py) translate their config.json into a spec and their tensors into the per-layer
 weight dicts ``load_layer`` takes; nothing below knows a family's names.
 
 One ``forward`` call runs a ragged batch: for every sequence its slot of the ``SequenceStateCache`` and its next
@@ -73,6 +74,8 @@ class SeqLayerSpec:
     taps: int = 1                     # short causal convolution on q and k
     bias: bool = False                # q, k, v projections carry biases
     head_bias: bool = False           # a number per head added to the scores
+    rot_pairs: str = "halves"         # which dimensions turn together: "halves": i and i + rot_dims / 2 | "neighbours": 2i and
+                                      # 2i + 1 (latent attention with direct queries)
     inv_freq: list | None = None      # rotary frequencies when they are not base^(-2i/rot_dims) (scaled forms)
     rot_mag: float = 1.0              # factor on cos and sin
     # cached attention, score options
@@ -87,6 +90,9 @@ class SeqLayerSpec:
     kv_from: int | None = None        # the layer has no key / value projections and reads that layer's keys and values
     # time mix (dim = vdim)
     decay_rank: int = 0
+    # gated delta rule (dim x vdim memories, kv_heads query / key heads, taps) and state-space memory (dim = state size, kv_heads =
+    # groups that share input and read-out vectors, norm_parts equal parts of the output normed on their own)
+    norm_parts: int = 1
     # a second mixer beside this one (pre-norm form): x += mix_scale * mixer + second_scale * second
     second: "SeqLayerSpec | None" = None
     mix_scale: float = 1.0
@@ -97,6 +103,7 @@ class SeqLayerSpec:
     form: str = "parallel"
     norm_offset: float = 0.0          # added to the layer's norm weights (1: weights stored around zero)
     norm_kind: str = "rms"            # pre-norm form: "rms" | "layer" (mean removed, weight and bias) | "dyt" (tanh(alpha x) w + b)
+    post_norm: bool = False           # pre-norm form: an RMS norm behind every block, x += norm(block output)
     layer_scale: bool = False         # pre-norm form: every block's output is multiplied by a learned vector
     residual_mult: float = 1.0        # pre-norm form: x += residual_mult * block output
     shift: bool = True
@@ -118,7 +125,19 @@ class SeqModelSpec:
     norm_kind: str = "rms"            # kind of the final norm (pre-norm form)
     pos_embed: str = ""               # "sinusoid": entry 2i of the embedding gets sin(p f_i), entry 2i + 1 cos(p f_i), ...
     pos_base: float = 10000.0         # ... f_i = pos_base^(-2i / width)
+    embed_norm: bool = False          # the embedding row passes an RMS norm with a weight of its own
+    loop: tuple | None = None         # (start, stop, times): layers start .. stop - 1 run `times` times in a row; in front of every
+                                      # pass x <- W [x; x0], x0 the embedding output
     eos_token_id: list = field(default_factory=list)
+
+    def layer_runs(self) -> list:
+        """[(layer, whether a pass of the loop begins in front of it)] in the order the layers run."""
+        n = len(self.layers)
+        if self.loop is None:
+            return [(i, False) for i in range(n)]
+        start, stop, times = self.loop
+        body = [(i, i == start) for i in range(start, stop)]
+        return [(i, False) for i in range(start)] + body * times + [(i, False) for i in range(stop, n)]
 
     # compatibility with the engines' view of a config
     @property
@@ -164,12 +183,24 @@ def rotary_inv_freq64(rot_dims: int, base: float) -> torch.Tensor:
 
 
 _MIXERS = {"retention": S.UMBS_MIX_RETENTION, "latent_attention": S.UMBS_MIX_LATENT_ATTENTION,
-           "cached_attention": S.UMBS_MIX_CACHED_ATTENTION, "mlstm": S.UMBS_MIX_MLSTM, "time_mix": S.UMBS_MIX_TIME_MIX}
+           "cached_attention": S.UMBS_MIX_CACHED_ATTENTION, "mlstm": S.UMBS_MIX_MLSTM, "time_mix": S.UMBS_MIX_TIME_MIX,
+           "gated_delta": S.UMBS_MIX_GATED_DELTA, "ssd": S.UMBS_MIX_SSD}
 _ATTN_MODES = {"softmax": S.UMBS_ATTN_SOFTMAX, "softmax_sink": S.UMBS_ATTN_SOFTMAX_SINK, "sigmoid": S.UMBS_ATTN_SIGMOID}
 _ACTS = {"clamped_glu": S.UMBS_ACT_CLAMPED_GLU, "gelu_tanh": S.UMBS_ACT_GELU_TANH, "silu": S.UMBS_ACT_SILU}
 _NORMS = {"rms": S.UMBS_NORM_RMS, "layer": S.UMBS_NORM_LAYER, "dyt": S.UMBS_NORM_DYT}
 _ROUTES = {"softmax_top": S.UMBS_ROUTE_SOFTMAX_TOP, "sigmoid_groups": S.UMBS_ROUTE_SIGMOID_GROUPS,
            "softmax_all": S.UMBS_ROUTE_SOFTMAX_ALL}
+
+
+def pair_rows_as_halves(w: torch.Tensor, first: int, rot_dims: int) -> torch.Tensor:
+    """Rows first .. first + rot_dims - 1 of ``w`` [..., rows, in], whose neighbours (2i, 2i + 1) turn together, reordered so that i
+    and i + rot_dims / 2 do: the kernels' pairing.  A score does not change when the dimensions of its query and its key are
+    reordered alike."""
+    n = w.shape[-2]
+    order = torch.arange(n, device=w.device)
+    r = torch.arange(first, first + rot_dims, device=w.device)
+    order[first:first + rot_dims] = torch.cat([r[0::2], r[1::2]])
+    return w.index_select(-2, order)
 
 
 def _softplus(z: float) -> float:
@@ -189,6 +220,13 @@ class SeqStateModel:
         self.model_name = model_name
         self.max_length = max_length
         self.num_layers = len(spec.layers)
+        self.runs = spec.layer_runs()
+        if spec.loop is not None:
+            start, stop, times = spec.loop
+            if not 0 <= start < stop <= self.num_layers or times < 1:
+                raise ValueError("loop: 0 <= start < stop <= layers and at least one pass")
+            if any(l.form != "prenorm" or l.kv_from is not None for l in spec.layers):
+                raise ValueError("a loop goes with pre-norm layers that keep their own keys and values")
         self.eos_tokens = list(spec.eos_token_id)
         self._slots0, self._max_tokens0 = slots, max_tokens
         self.weights: list[dict | None] = [None] * self.num_layers
@@ -234,13 +272,21 @@ class SeqStateModel:
         return t.to(self.device, torch.float32).contiguous()
 
     def load_head(self, embed: torch.Tensor, head: torch.Tensor | None, final_norm: torch.Tensor,
-                  final_norm_b: torch.Tensor | None = None, final_norm_alpha: float = 1.0):
-        """``head`` None: the logits come from the embedding table itself (tied)."""
+                  final_norm_b: torch.Tensor | None = None, final_norm_alpha: float = 1.0, embed_norm: torch.Tensor | None = None,
+                  loop_in: torch.Tensor | None = None):
+        """``head`` None: the logits come from the embedding table itself (tied).  ``embed_norm`` [width], ``loop_in`` [width,
+        2 width] (columns for x, then for the embedding output): the embedding's norm and the product in front of a loop's passes."""
         e = self._act(embed)
         self.head_weights = dict(embed=e, head=e if head is None else self._act(head), final_norm=self._f32(final_norm))
         if self.spec.norm_kind in ("layer", "dyt"):
             self.head_weights["final_norm_b"] = self._f32(final_norm_b)
         self.final_norm_alpha = float(final_norm_alpha)
+        if self.spec.embed_norm:
+            self.head_weights["embed_norm"] = self._f32(embed_norm)
+            assert self.head_weights["embed_norm"].numel() == self.spec.width
+        if self.spec.loop is not None:
+            self.head_weights["loop_in"] = self._act(loop_in)
+            assert self.head_weights["loop_in"].shape == (self.spec.width, 2 * self.spec.width)
         if self.spec.pos_embed == "sinusoid":
             self.head_weights["pos_freq"] = rotary_inv_freq(self.spec.width, self.spec.pos_base).to(self.device)
         elif self.spec.pos_embed:
@@ -259,7 +305,11 @@ class SeqStateModel:
         mlstm: q, k [heads dim, width]; v, g [heads vdim, width]; i, f [heads, width] with i_b, f_b [heads]; out_norm [heads vdim].
         latent attention with direct queries (q_rank 0): q [heads (dim + rope_dim), width], dkv [kv_rank + rope_dim, width],
             dkv_norm, uk, uv, g [heads vdim, width] (gate_kind 2), sink [heads] (learned_sink).
-        pre-norm layers: norm2 [width] when they have a feed-forward; norm_b, norm2_b (layer norm); ls1, ls2 [width] (layer scale).
+        gated delta: q, k [kv_heads dim, width]; v, g [heads vdim, width]; b, a [heads, width]; q_conv, k_conv, v_conv [channels, taps];
+            A_log, dt_bias [heads]; out_norm [vdim].
+        state space: in [2 heads vdim + 2 kv_heads dim + heads, width] (gate | v | k | q | step size); conv [channels of v | k | q, taps],
+            conv_b; A_log, dt_bias, D [heads]; out_norm [heads vdim].
+        pre-norm layers: post_norm, post_norm2 [width] (norms behind the blocks); norm2 [width] when they have a feed-forward; norm_b, norm2_b (layer norm); ls1, ls2 [width] (layer scale).
         feed-forward: router [experts, width]; experts: list of (gate, up, down); shared (or dense): (gate, up, down);
             dense_b: (gate_b, up_b, down_b) with ``bias``; shared_gate [1, width] or [width]."""
         l = self.spec.layers[idx]
@@ -275,6 +325,10 @@ class SeqStateModel:
             if l.norm_kind == "dyt":           # the scalars inside the tanh
                 d["norm_alpha"] = float(w["norm_alpha"])
                 d["norm2_alpha"] = float(w["norm2_alpha"]) if l.mlp is not None else 1.0
+            if l.post_norm:
+                d["post_norm"] = self._f32(w["post_norm"])
+                if l.mlp is not None:
+                    d["post_norm2"] = self._f32(w["post_norm2"])
             if l.layer_scale:
                 d["ls1"] = self._f32(w["ls1"])
                 if l.mlp is not None:
@@ -308,7 +362,13 @@ class SeqStateModel:
             if l.form != "prenorm":
                 raise ValueError("latent attention with direct queries is a pre-norm mixer")
             hd1 = l.dim + l.rope_dim
-            d["w_in"] = self._act(torch.cat([w["q"], w["dkv"]] + ([w["g"]] if l.gate_kind else []), dim=0))
+            wq, wdkv = w["q"], w["dkv"]
+            if l.rot_pairs == "neighbours" and l.rot_dims:
+                wq = pair_rows_as_halves(wq.reshape(l.heads, hd1, -1), l.dim, l.rot_dims).reshape(wq.shape)
+                wdkv = pair_rows_as_halves(wdkv, l.kv_rank, l.rot_dims)
+            elif l.rot_pairs not in ("halves", "neighbours"):
+                raise ValueError(f"unknown rotary pairing '{l.rot_pairs}'")
+            d["w_in"] = self._act(torch.cat([wq, wdkv] + ([w["g"]] if l.gate_kind else []), dim=0))
             d["kv_norm"] = self._f32(w["dkv_norm"])
             d["ukT"] = self._act(w["uk"].reshape(l.heads, l.dim, l.kv_rank).transpose(1, 2))
             d["uv"] = self._act(w["uv"])
@@ -382,6 +442,24 @@ class SeqStateModel:
             l.decay_rank = int(w["w1"].shape[0])
             assert l.vdim == l.dim and d["w_in"].shape == (4, hd, self.spec.width) and d["mu"].shape == (5, self.spec.width)
             assert d["w2"].shape == (hd, l.decay_rank) and d["w0"].numel() == hd and d["u"].numel() == hd and d["out_norm"].numel() == hd
+        elif l.mixer in ("gated_delta", "ssd"):
+            hv, gd = l.heads * l.vdim, l.kv_heads * l.dim
+            if l.form != "prenorm" or l.heads % l.kv_heads:
+                raise ValueError("rank-one memories are pre-norm mixers whose heads share their query / key heads evenly")
+            if l.mixer == "gated_delta":
+                d["w_in"] = self._act(torch.cat([w["q"], w["k"], w["v"], w["g"], w["b"], w["a"]], dim=0))
+                d["conv_w"] = self._f32(torch.cat([w["q_conv"], w["k_conv"], w["v_conv"]], dim=0))
+                assert d["w_in"].shape == (2 * gd + 2 * hv + 2 * l.heads, self.spec.width)
+            else:
+                d["w_in"], d["conv_w"], d["conv_b"] = self._act(w["in"]), self._f32(w["conv"]), self._f32(w["conv_b"])
+                d["skip"] = self._f32(w["D"])
+                assert d["w_in"].shape == (2 * hv + 2 * gd + l.heads, self.spec.width) and d["conv_b"].numel() == 2 * gd + hv
+                assert hv % l.norm_parts == 0 and d["skip"].numel() == l.heads
+            # the decay's rate exp(A_log), evaluated once in double
+            d["decay_rate"], d["dt_bias"] = self._f32(torch.exp(w["A_log"].double())), self._f32(w["dt_bias"])
+            d["out_norm"] = self._f32(w["out_norm"])
+            assert d["conv_w"].shape == (2 * gd + hv, l.taps) and d["decay_rate"].numel() == l.heads and d["dt_bias"].numel() == l.heads
+            assert d["out_norm"].numel() == (l.vdim if l.mixer == "gated_delta" else hv)
         elif l.mixer == "mlstm":
             d["w_in"] = self._act(torch.cat([w["q"], w["k"], w["v"], w["g"], w["i"], w["f"]], dim=0))
             d["bias_in"] = self._f32(torch.cat([w["i_b"], w["f_b"]]))
@@ -444,7 +522,7 @@ class SeqStateModel:
         assert self.head_weights is not None and all(w is not None for w in self.weights), "load every layer first"
         sp, cache = self.spec, self.cache
         p = lambda t: t.data_ptr() if t is not None else None
-        layers = (S.Layer * self.num_layers)()
+        layers = (S.Layer * len(self.runs))()
         seconds = []
 
         def fill_mixer(cl, l, w, i):
@@ -475,6 +553,11 @@ class SeqStateModel:
                 cl.mix_mu, cl.decay_rank, cl.w_decay1, cl.w_decay2 = p(w["mu"]), l.decay_rank, p(w["w1"]), p(w["w2"])
                 cl.decay_bias, cl.bonus, cl.out_norm_w = p(w["w0"]), p(w["u"]), p(w["out_norm"])
                 cl.tm_state, cl.shift_state = p(cache.tm_state[i]), p(cache.shift[i])
+            elif l.mixer in ("gated_delta", "ssd"):
+                cl.kv_heads, cl.taps, cl.norm_parts = l.kv_heads, l.taps, l.norm_parts
+                cl.conv_w, cl.conv_b, cl.conv_state = p(w["conv_w"]), p(w.get("conv_b")), p(cache.conv_state[i])
+                cl.decay_rate, cl.dt_bias, cl.skip_w = p(w["decay_rate"]), p(w["dt_bias"]), p(w.get("skip"))
+                cl.out_norm_w, cl.mem_state = p(w["out_norm"]), p(cache.mem_state[i])
             elif l.mixer == "mlstm":
                 cl.gate_cap, cl.bias_in, cl.out_norm_w = l.gate_cap, p(w["bias_in"]), p(w["out_norm"])
                 cl.mlstm_state = p(cache.mlstm_state[i])
@@ -490,13 +573,16 @@ class SeqStateModel:
                     cl.attn_mode, cl.gate_kind, cl.sink = _ATTN_MODES[l.attn_mode], l.gate_kind, p(w.get("sink"))
             cl.w_in, cl.w_o = p(w["w_in"]), p(w["o"])
 
-        for i, (l, w) in enumerate(zip(sp.layers, self.weights)):
-            cl = layers[i]
+        for i, (li, begins) in enumerate(self.runs):           # one struct per layer run: shared weights, state of its own
+            l, w, cl = sp.layers[li], self.weights[li], layers[i]
+            if begins:
+                cl.w_merge = p(self.head_weights["loop_in"])
             fill_mixer(cl, l, w, i)
             cl.form = S.UMBS_FORM_PRENORM if l.form == "prenorm" else S.UMBS_FORM_PARALLEL
             cl.norm_offset, cl.norm2_w = l.norm_offset, p(w.get("norm2"))
             cl.norm_kind, cl.norm_b, cl.norm2_b = _NORMS[l.norm_kind], p(w.get("norm_b")), p(w.get("norm2_b"))
             cl.norm_alpha, cl.norm2_alpha = w.get("norm_alpha", 1.0), w.get("norm2_alpha", 1.0)
+            cl.post_norm_w, cl.post_norm2_w = p(w.get("post_norm")), p(w.get("post_norm2"))
             cl.out_scale, cl.out_scale2, cl.residual_mult = p(w.get("ls1")), p(w.get("ls2")), l.residual_mult
             cl.norm_w = p(w["norm"])
             if l.mixer != "time_mix":
@@ -504,7 +590,7 @@ class SeqStateModel:
             cl.depth_w = p(w.get("depth"))
             if l.second is not None:
                 sec = S.Layer()
-                fill_mixer(sec, l.second, w["second"], l.second.state_index)
+                fill_mixer(sec, l.second, w["second"], cache.second_index[i])
                 seconds.append(sec)
                 cl.second, cl.mix_scale, cl.second_scale = C.pointer(sec), l.mix_scale, l.second_scale
             cl.has_mlp = int(l.mlp is not None)
@@ -524,12 +610,13 @@ class SeqStateModel:
                     cl.mlp.unary_p0, cl.mlp.unary_p1 = w["unary_p"]
         m = S.Model()
         m.dtype = S.UMBS_BF16 if self.dtype == torch.bfloat16 else S.UMBS_F32
-        m.width, m.vocab, m.n_layers, m.norm_groups, m.slots = sp.width, sp.vocab, self.num_layers, sp.norm_groups, cache.slots
+        m.width, m.vocab, m.n_layers, m.norm_groups, m.slots = sp.width, sp.vocab, len(self.runs), sp.norm_groups, cache.slots
         m.norm_eps, m.norm_offset, m.logit_softcap = sp.norm_eps, sp.norm_offset, sp.logit_softcap
         hw = self.head_weights
         m.embed, m.final_norm, m.head = p(hw["embed"]), p(hw["final_norm"]), p(hw["head"])
         m.embed_scale, m.norm_kind, m.final_norm_b = sp.embed_scale, _NORMS[sp.norm_kind], p(hw.get("final_norm_b"))
         m.final_norm_alpha, m.pos_freq = getattr(self, "final_norm_alpha", 1.0), p(hw.get("pos_freq"))
+        m.embed_norm = p(hw.get("embed_norm"))
         m.layers = C.cast(layers, C.POINTER(S.Layer))
         self._c_layers = (layers, seconds)
         self._c_model, self._c_version = m, self.cache.version
@@ -540,7 +627,7 @@ class SeqStateModel:
     def forward(self, entries, layer_out: bool = False):
         """``entries``: [(slot, tokens, want)], the next tokens of every sequence of the step and the indices among
         them whose logits are wanted.  Returns fp32 logits [sum of wants, vocab] in entry order (and, with
-        ``layer_out``, the residual stream after every layer, [layers, tokens, width]).  The slots' positions advance."""
+        ``layer_out``, the residual stream after every layer run, [runs, tokens, width]).  The slots' positions advance."""
         cache = self.cache
         ids, tok_seq, tok_pos, want = [], [], [], []
         slot, start, length, pos0, parity = [], [], [], [], []
@@ -590,7 +677,7 @@ class SeqStateModel:
         if logits is None:
             dev = host.to(self.device, non_blocking=True)
             logits = torch.empty((Wn, self.spec.vocab), dtype=torch.float32, device=self.device)
-            layers = torch.empty((self.num_layers, T, self.spec.width), dtype=torch.float32, device=self.device) \
+            layers = torch.empty((len(self.runs), T, self.spec.width), dtype=torch.float32, device=self.device) \
                 if layer_out else None
             enqueue(describe(dev.data_ptr()), logits, layers)
             self._keep = (host, dev)          # alive until the next step is enqueued behind this one
