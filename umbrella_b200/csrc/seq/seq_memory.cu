@@ -26,86 +26,159 @@ __device__ __forceinline__ float softplus_mem(float z) { return fmaxf(z, 0.f) + 
 constexpr int kPrepWarps = 4, kPrepVals = 4;       // warps per block; channels per lane of a value task
 
 // A warp's task: one query / key head (both vectors, their norms and their dot product), 128 value channels, or the gates
-// of all heads -- for `tile` consecutive tokens, so that the rows a convolution shares with its neighbours are read through
-// L1.  A lane's sums run in a fixed order, so a token's result does not depend on what else is in the step.
-template <int NC>
+// of all heads -- for TT consecutive tokens.  TAPS > 0: the number of taps is known, the tile's projected values and the
+// rows in front of it are loaded into registers together and every convolution reads them there; TAPS == 0: any number, one
+// value at a time.  A lane's sums run in a fixed order, so a token's result does not depend on what else is in the step.
+template <int NC, int TAPS, int TT>
 __global__ void __launch_bounds__(32 * kPrepWarps) memory_prep_kernel(const float* __restrict__ proj, int64_t ld, umbs_memory_t m, Batch b,
-                                                                      int slots, int tile, float* __restrict__ qkv, int64_t ld_qkv,
+                                                                      int slots, float* __restrict__ qkv, int64_t ld_qkv,
                                                                       float* __restrict__ gates, float* __restrict__ kq) {
     const int lane = threadIdx.x & 31, task = blockIdx.y * kPrepWarps + (threadIdx.x >> 5);
-    const int G = m.kv_heads, D = m.dim, cv = m.heads * m.vdim, C = 2 * G * D + cv, taps = m.taps, keep = taps - 1;
+    const int G = m.kv_heads, D = m.dim, cv = m.heads * m.vdim, C = 2 * G * D + cv, taps = TAPS > 0 ? TAPS : m.taps, keep = taps - 1;
     const int vtasks = (cv + 32 * kPrepVals - 1) / (32 * kPrepVals);
+    const int t0 = blockIdx.x * TT, nt = min(TT, b.n_tokens - t0);
     if (task > G + vtasks) return;
-    const int t_end = min(b.n_tokens, (int)(blockIdx.x + 1) * tile);
-    for (int t = blockIdx.x * tile; t < t_end; ++t) {
-        if (task == G + vtasks) {
+    if (task == G + vtasks) {
+        for (int i = lane; i < nt * m.heads; i += 32) {
+            const int t = t0 + i / m.heads, h = i % m.heads;
             const float* row = proj + (int64_t)t * ld;
-            for (int h = lane; h < m.heads; h += 32) {
-                const float dt = softplus_mem(row[m.off_decay + h] + m.dt_bias[h]);
-                float* g = gates + ((int64_t)t * m.heads + h) * 2;
-                g[0] = -m.decay_rate[h] * dt;
-                g[1] = m.off_strength >= 0 ? 1.f / (1.f + expf(-row[m.off_strength + h])) : dt;
-            }
-            continue;
+            const float dt = softplus_mem(row[m.off_decay + h] + m.dt_bias[h]);
+            float* g = gates + ((int64_t)t * m.heads + h) * 2;
+            g[0] = -m.decay_rate[h] * dt;
+            g[1] = m.off_strength >= 0 ? 1.f / (1.f + expf(-row[m.off_strength + h])) : dt;
         }
-        const int s = b.tok_seq[t], pos = b.tok_pos[t];
-        const int start = b.seq_start[s], len = b.seq_len[s], pos0 = b.seq_pos0[s], slot = b.seq_slot[s], par = b.seq_parity[s];
-        const float* st_in = keep > 0 ? m.conv_state + ((int64_t)par * slots + slot) * keep * C : nullptr;
-        // the projected value of channel c at position p: this step's row, the carried rows, or zero in front of the sequence
-        auto u_at = [&](int c, int p) -> float {
-            if (p >= pos0) return proj[(int64_t)(start + p - pos0) * ld + m.off_conv + c];
-            return p < 0 ? 0.f : st_in[(int64_t)(p - (pos0 - keep)) * C + c];
-        };
-        auto conv = [&](int c) -> float {
-            float acc = m.conv_b != nullptr ? m.conv_b[c] : 0.f;
-            for (int j = 0; j < taps; ++j) acc = fmaf(m.conv_w[(int64_t)c * taps + j], u_at(c, pos - keep + j), acc);
-            return silu_mem(acc);
-        };
-        // the sequence's last token of the step leaves the rows the next step starts from (the other half of the buffer)
-        const bool last = keep > 0 && t == start + len - 1;
-        float* st_out = last ? m.conv_state + ((int64_t)(par ^ 1) * slots + slot) * keep * C : nullptr;
-        auto carry = [&](int c) {
-            for (int r = 0; r < keep; ++r) st_out[(int64_t)r * C + c] = u_at(c, pos0 + len - keep + r);
-        };
-        float* out = qkv + (int64_t)t * ld_qkv;
-        if (task < G) {
-            const int cq = m.off_q + task * D, ck = m.off_k + task * D;
-            float q[NC], k[NC], qq = 0.f, kk = 0.f, dot = 0.f;
+        return;
+    }
+    int start[TT], pos0[TT];                       // per token: first row of its sequence in the step, position of that row
+    int64_t st_in[TT];                             // where its sequence's carried rows begin
+    bool last[TT];
+#pragma unroll
+    for (int j = 0; j < TT; ++j) {
+        const int s = j < nt ? b.tok_seq[t0 + j] : b.tok_seq[t0];
+        start[j] = b.seq_start[s];
+        pos0[j] = b.seq_pos0[s];
+        st_in[j] = ((int64_t)b.seq_parity[s] * slots + b.seq_slot[s]) * keep * C;
+        last[j] = keep > 0 && j < nt && t0 + j == start[j] + b.seq_len[s] - 1;
+    }
+    // channel c of the row `back` rows in front of the first row of token j's sequence: a carried row, or zero in front of the sequence
+    auto carried = [&](int j, int c, int back) -> float {
+        return pos0[j] >= back ? m.conv_state[st_in[j] + (int64_t)(keep - back) * C + c] : 0.f;
+    };
+    // the other half of the buffer: the sequence's last token of the step leaves the rows the next step starts from
+    auto carry_slot = [&](int j) -> float* {
+        const int s = b.tok_seq[t0 + j];
+        return m.conv_state + ((int64_t)(b.seq_parity[s] ^ 1) * slots + b.seq_slot[s]) * keep * C;
+    };
+    constexpr int KEEP = TAPS > 1 ? TAPS - 1 : 0, ROWS = TAPS > 0 ? TT + KEEP : 1;
+    // One channel: raw[] are its projected values at rows t0 - KEEP .. t0 + TT - 1 of the step.
+    auto fetch = [&](int c, float (&raw)[ROWS]) {
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int r = 0; r < ROWS; ++r) {
+                const int t = t0 - KEEP + r;
+                raw[r] = (t >= 0 && t < t0 + nt) ? proj[(int64_t)t * ld + m.off_conv + c] : 0.f;
+            }
+        }
+    };
+    auto conv = [&](int j, int c, const float (&raw)[ROWS], const float (&w)[TAPS > 0 ? TAPS : 1], float bias) -> float {
+        float acc = bias;
+        const int r0 = t0 + j - start[j];          // the token's row in its sequence's part of the step
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int x = 0; x < TAPS; ++x) {
+                const int r = r0 - KEEP + x;
+                acc = fmaf(w[x], r >= 0 ? raw[j + x] : carried(j, c, -r), acc);
+            }
+        } else {
+            for (int x = 0; x < taps; ++x) {
+                const int r = r0 - keep + x;
+                acc = fmaf(m.conv_w[(int64_t)c * taps + x], r >= 0 ? proj[(int64_t)(start[j] + r) * ld + m.off_conv + c] : carried(j, c, -r), acc);
+            }
+        }
+        return silu_mem(acc);
+    };
+    auto carry = [&](int j, int c, const float (&raw)[ROWS]) {
+        float* out = carry_slot(j);
+        const int r0 = t0 + j - start[j];
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int x = 0; x < KEEP; ++x) {
+                const int r = r0 - KEEP + 1 + x;
+                out[(int64_t)x * C + c] = r >= 0 ? raw[j + 1 + x] : carried(j, c, -r);
+            }
+        } else {
+            for (int x = 0; x < keep; ++x) {
+                const int r = r0 - keep + 1 + x;
+                out[(int64_t)x * C + c] = r >= 0 ? proj[(int64_t)(start[j] + r) * ld + m.off_conv + c] : carried(j, c, -r);
+            }
+        }
+    };
+    auto weights = [&](int c, float (&w)[TAPS > 0 ? TAPS : 1]) -> float {
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int x = 0; x < TAPS; ++x) w[x] = m.conv_w[(int64_t)c * TAPS + x];
+        }
+        return m.conv_b != nullptr ? m.conv_b[c] : 0.f;
+    };
+    if (task < G) {
+        // the head's query, then its key: convolved values of the whole tile in registers, then the norms and the dot product
+        float y[2][TT][NC];
+#pragma unroll
+        for (int v = 0; v < 2; ++v) {
+            const int c0 = (v == 0 ? m.off_q : m.off_k) + task * D;
 #pragma unroll
             for (int i = 0; i < NC; ++i) {
-                const int d = lane + 32 * i;
-                q[i] = k[i] = 0.f;
-                if (d < D) {
-                    q[i] = conv(cq + d);
-                    k[i] = conv(ck + d);
-                    qq = fmaf(q[i], q[i], qq);
-                    kk = fmaf(k[i], k[i], kk);
-                    if (last) { carry(cq + d); carry(ck + d); }
+                const int d = lane + 32 * i, c = c0 + d;
+#pragma unroll
+                for (int j = 0; j < TT; ++j) y[v][j][i] = 0.f;
+                if (d >= D) continue;
+                float raw[ROWS], w[TAPS > 0 ? TAPS : 1];
+                fetch(c, raw);
+                const float bias = weights(c, w);
+#pragma unroll
+                for (int j = 0; j < TT; ++j) {
+                    if (j >= nt) break;
+                    y[v][j][i] = conv(j, c, raw, w, bias);
+                    if (last[j]) carry(j, c, raw);
                 }
             }
-            float fq = 1.f, fk = 1.f;
+        }
+#pragma unroll
+        for (int j = 0; j < TT; ++j) {
+            if (j >= nt) break;
+            float fq = 1.f, fk = 1.f, dot = 0.f;
             if (m.unit) {
+                float qq = 0.f, kk = 0.f;
+#pragma unroll
+                for (int i = 0; i < NC; ++i) { qq = fmaf(y[0][j][i], y[0][j][i], qq); kk = fmaf(y[1][j][i], y[1][j][i], kk); }
                 fq = 1.f / sqrtf(warp_sum_mem(qq) + 1e-6f) * (1.f / sqrtf((float)D));
                 fk = 1.f / sqrtf(warp_sum_mem(kk) + 1e-6f);
             }
+            float* out = qkv + (int64_t)(t0 + j) * ld_qkv;
 #pragma unroll
             for (int i = 0; i < NC; ++i) {
                 const int d = lane + 32 * i;
-                q[i] *= fq;
-                k[i] *= fk;
-                dot = fmaf(q[i], k[i], dot);
-                if (d < D) { out[cq + d] = q[i]; out[ck + d] = k[i]; }
+                const float q = y[0][j][i] * fq, k = y[1][j][i] * fk;
+                dot = fmaf(q, k, dot);
+                if (d < D) { out[m.off_q + task * D + d] = q; out[m.off_k + task * D + d] = k; }
             }
             dot = warp_sum_mem(dot);
-            if (lane == 0) kq[(int64_t)t * G + task] = dot;
-        } else {
-            const int c0 = (task - G) * 32 * kPrepVals;
+            if (lane == 0) kq[(int64_t)(t0 + j) * G + task] = dot;
+        }
+    } else {
+        const int c0 = (task - G) * 32 * kPrepVals;
 #pragma unroll
-            for (int i = 0; i < kPrepVals; ++i) {
-                const int c = c0 + lane + 32 * i;
-                if (c >= cv) continue;
-                out[m.off_v + c] = conv(m.off_v + c);
-                if (last) carry(m.off_v + c);
+        for (int i = 0; i < kPrepVals; ++i) {
+            const int e = c0 + lane + 32 * i, c = m.off_v + e;
+            if (e >= cv) continue;
+            float raw[ROWS], w[TAPS > 0 ? TAPS : 1];
+            fetch(c, raw);
+            const float bias = weights(c, w);
+#pragma unroll
+            for (int j = 0; j < TT; ++j) {
+                if (j >= nt) break;
+                qkv[(int64_t)(t0 + j) * ld_qkv + c] = conv(j, c, raw, w, bias);
+                if (last[j]) carry(j, c, raw);
             }
         }
     }
@@ -166,40 +239,45 @@ __global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __r
     // rows beyond dim and columns beyond vdim of every stage stay zero
     for (int i = tid; i < kMemStages * STAGE; i += 32 * kMemWarps) mem_sm[i] = 0.f;
     __syncthreads();
+    constexpr int NT = 32 * kMemWarps, P4 = DP / 4, C4 = CT / 4;
     auto issue = [&](int g) {
         float* sq = mem_sm + (g % kMemStages) * STAGE;
         float* sk = sq + TB * DP;
         float* sv = sk + TB * DP;
-        float* sg = sv + TB * CT;                                                  // [3][TB] decay, strength, k . q
+        float* sg = sv + TB * CT;                                                  // [TB][4] decay, strength, k . q
         const int t0 = g * TB, nt = min(TB, len - t0);
         const float* base = qkv + (int64_t)(start + t0) * ld;
         if (vec) {
-            const int p = D / 4;
-            for (int i = tid; i < nt * p; i += 32 * kMemWarps) {
-                const int tt = i / p, d = (i - tt * p) * 4;
-                cp_async16(sq + tt * DP + d, base + (int64_t)tt * ld + cq + d);
-                cp_async16(sk + tt * DP + d, base + (int64_t)tt * ld + ck + d);
+#pragma unroll
+            for (int i = tid; i < TB * P4; i += NT) {
+                const int tt = i / P4, d = (i % P4) * 4;
+                if (tt < nt && d < D) {
+                    cp_async16(sq + tt * DP + d, base + (int64_t)tt * ld + cq + d);
+                    cp_async16(sk + tt * DP + d, base + (int64_t)tt * ld + ck + d);
+                }
             }
-            for (int i = tid; i < nt * (CT / 4); i += 32 * kMemWarps) {
-                const int tt = i / (CT / 4), d = (i - tt * (CT / 4)) * 4;
-                if (d < ncol) cp_async16(sv + tt * CT + d, base + (int64_t)tt * ld + cv + d);
+            for (int i = tid; i < TB * C4; i += NT) {
+                const int tt = i / C4, d = (i % C4) * 4;
+                if (tt < nt && d < ncol) cp_async16(sv + tt * CT + d, base + (int64_t)tt * ld + cv + d);
             }
         } else {
-            for (int i = tid; i < nt * D; i += 32 * kMemWarps) {
-                const int tt = i / D, d = i - tt * D;
-                cp_async4(sq + tt * DP + d, base + (int64_t)tt * ld + cq + d);
-                cp_async4(sk + tt * DP + d, base + (int64_t)tt * ld + ck + d);
+            for (int i = tid; i < TB * DP; i += NT) {
+                const int tt = i / DP, d = i % DP;
+                if (tt < nt && d < D) {
+                    cp_async4(sq + tt * DP + d, base + (int64_t)tt * ld + cq + d);
+                    cp_async4(sk + tt * DP + d, base + (int64_t)tt * ld + ck + d);
+                }
             }
-            for (int i = tid; i < nt * CT; i += 32 * kMemWarps) {
-                const int tt = i / CT, d = i - tt * CT;
-                if (d < ncol) cp_async4(sv + tt * CT + d, base + (int64_t)tt * ld + cv + d);
+            for (int i = tid; i < TB * CT; i += NT) {
+                const int tt = i / CT, d = i % CT;
+                if (tt < nt && d < ncol) cp_async4(sv + tt * CT + d, base + (int64_t)tt * ld + cv + d);
             }
         }
         if (tid < nt) {
             const int64_t t = start + t0 + tid;
-            cp_async4(sg + tid, gates + (t * m.heads + h) * 2);
-            cp_async4(sg + TB + tid, gates + (t * m.heads + h) * 2 + 1);
-            cp_async4(sg + 2 * TB + tid, kq + t * m.kv_heads + grp);
+            cp_async4(sg + 4 * tid, gates + (t * m.heads + h) * 2);
+            cp_async4(sg + 4 * tid + 1, gates + (t * m.heads + h) * 2 + 1);
+            cp_async4(sg + 4 * tid + 2, kq + t * m.kv_heads + grp);
         }
     };
     const int groups = (len + TB - 1) / TB;
@@ -217,48 +295,58 @@ __global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __r
         float* sv = sk + TB * DP;
         float* sg = sv + TB * CT;
         const int t0 = g * TB, nt = min(TB, len - t0);
-        if (tid < nt) sg[tid] = expf(sg[tid]);                                     // (the thread that copied it)
+        if (tid < nt) sg[4 * tid] = expf(sg[4 * tid]);                             // (the thread that copied it)
         __syncthreads();
-        for (int tt = 0; tt < nt; ++tt) {
-            const float dec = sg[tt], str = sg[TB + tt], dot = sg[2 * TB + tt];
-            float k[RPL], aq[CPL][4], ak[CPL][4];
-#pragma unroll
-            for (int c = 0; c < CPL; ++c)
-#pragma unroll
-                for (int x = 0; x < 4; ++x) aq[c][x] = ak[c][x] = 0.f;
+        // the operands of a token are in registers before the token in front of it is worked on
+        struct Operands { float k[RPL], q[RPL], v[CPL]; float4 g; } op[2];
+        auto load = [&](Operands& x, int tt) {
+            x.g = *reinterpret_cast<const float4*>(sg + 4 * tt);
 #pragma unroll
             for (int i = 0; i < RPL / 4; ++i) {
                 const float4 k4 = *reinterpret_cast<const float4*>(sk + tt * DP + 4 * (rl + RL * i));
                 const float4 q4 = *reinterpret_cast<const float4*>(sq + tt * DP + 4 * (rl + RL * i));
-                k[4 * i] = k4.x; k[4 * i + 1] = k4.y; k[4 * i + 2] = k4.z; k[4 * i + 3] = k4.w;
-                const float qa[4] = {q4.x, q4.y, q4.z, q4.w};
-#pragma unroll
-                for (int c = 0; c < CPL; ++c)
-#pragma unroll
-                    for (int x = 0; x < 4; ++x) {
-                        if (DELTA) ak[c][x] = fmaf(S[c][4 * i + x], k[4 * i + x], ak[c][x]);
-                        aq[c][x] = fmaf(S[c][4 * i + x], qa[x], aq[c][x]);
-                    }
+                x.k[4 * i] = k4.x; x.k[4 * i + 1] = k4.y; x.k[4 * i + 2] = k4.z; x.k[4 * i + 3] = k4.w;
+                x.q[4 * i] = q4.x; x.q[4 * i + 1] = q4.y; x.q[4 * i + 2] = q4.z; x.q[4 * i + 3] = q4.w;
             }
 #pragma unroll
+            for (int c = 0; c < CPL; ++c) x.v[c] = sv[tt * CT + col[c]];
+        };
+        auto walk = [&](const Operands& x, int tt) {
+            const float dec = x.g.x, str = x.g.y, dot = x.g.z;
+#pragma unroll
             for (int c = 0; c < CPL; ++c) {
-                float dq = (aq[c][0] + aq[c][1]) + (aq[c][2] + aq[c][3]);
-                float dk = (ak[c][0] + ak[c][1]) + (ak[c][2] + ak[c][3]);
+                float aq[4] = {0.f, 0.f, 0.f, 0.f}, ak[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int i = 0; i < RPL; i += 4)
+#pragma unroll
+                    for (int y = 0; y < 4; ++y) {
+                        if (DELTA) ak[y] = fmaf(S[c][i + y], x.k[i + y], ak[y]);
+                        aq[y] = fmaf(S[c][i + y], x.q[i + y], aq[y]);
+                    }
+                float dq = (aq[0] + aq[1]) + (aq[2] + aq[3]);
+                float dk = (ak[0] + ak[1]) + (ak[2] + ak[3]);
 #pragma unroll
                 for (int w = RL / 2; w > 0; w >>= 1) {
                     if (DELTA) dk += __shfl_xor_sync(0xffffffffu, dk, w);
                     dq += __shfl_xor_sync(0xffffffffu, dq, w);
                 }
-                const float v = sv[tt * CT + col[c]];
-                const float u = DELTA ? str * fmaf(-dec, dk, v) : str * v;
+                const float u = DELTA ? str * fmaf(-dec, dk, x.v[c]) : str * x.v[c];
 #pragma unroll
-                for (int i = 0; i < RPL; ++i) S[c][i] = fmaf(dec, S[c][i], k[i] * u);
-                if (rl == 0) so[tt * CT + col[c]] = fmaf(skip, v, fmaf(dot, u, dec * dq));
+                for (int i = 0; i < RPL; ++i) S[c][i] = fmaf(dec, S[c][i], x.k[i] * u);
+                if (rl == 0) so[tt * CT + col[c]] = fmaf(skip, x.v[c], fmaf(dot, u, dec * dq));
             }
+        };
+        load(op[0], 0);
+        for (int tt = 0; tt < nt; tt += 2) {
+            load(op[1], tt + 1);                                                   // (TB is even: a place of the stage)
+            walk(op[0], tt);
+            if (tt + 1 >= nt) break;
+            load(op[0], min(tt + 2, TB - 1));
+            walk(op[1], tt + 1);
         }
         __syncthreads();
-        for (int i = tid; i < nt * CT; i += 32 * kMemWarps) {
-            const int tt = i / CT, c = i - tt * CT;
+        for (int i = tid; i < nt * CT; i += NT) {
+            const int tt = i / CT, c = i % CT;
             if (c < ncol) o[(int64_t)(start + t0 + tt) * hv + h * V + c0 + c] = so[i];
         }
     }
@@ -345,11 +433,23 @@ extern "C" int umbs_memory_prep(const float* proj, int64_t ld, const umbs_memory
         return UMB_ERR_ARG;
     cudaStream_t st = (cudaStream_t)stream;
     const int tasks = m->kv_heads + (m->heads * m->vdim + 32 * kPrepVals - 1) / (32 * kPrepVals) + 1;
-    const int tile = batch->n_tokens > 256 ? 8 : 1;
+    // a long step: tiles of consecutive tokens, as long as the registers of a head's size allow
+    const bool wide = batch->n_tokens > 256 && m->taps == 4;
+    const int nc = m->dim <= 64 ? 2 : (m->dim <= 128 ? 4 : (m->dim <= 256 ? 8 : 16)), tile = wide ? 16 / nc : 1;
     const dim3 grid((batch->n_tokens + tile - 1) / tile, (tasks + kPrepWarps - 1) / kPrepWarps);
-    if (m->dim <= 64) memory_prep_kernel<2><<<grid, 32 * kPrepWarps, 0, st>>>(proj, ld, *m, *batch, slots, tile, qkv, ld_qkv, gates, kq);
-    else if (m->dim <= 128) memory_prep_kernel<4><<<grid, 32 * kPrepWarps, 0, st>>>(proj, ld, *m, *batch, slots, tile, qkv, ld_qkv, gates, kq);
-    else memory_prep_kernel<16><<<grid, 32 * kPrepWarps, 0, st>>>(proj, ld, *m, *batch, slots, tile, qkv, ld_qkv, gates, kq);
+#define UMBS_PREP(NC, TAPS, TT) memory_prep_kernel<NC, TAPS, TT><<<grid, 32 * kPrepWarps, 0, st>>>(proj, ld, *m, *batch, slots, qkv, ld_qkv, gates, kq)
+#define UMBS_PREP_NC(NC)                              \
+    do {                                              \
+        if (wide) UMBS_PREP(NC, 4, 16 / NC);          \
+        else if (m->taps == 4) UMBS_PREP(NC, 4, 1);   \
+        else UMBS_PREP(NC, 0, 1);                     \
+    } while (0)
+    if (nc == 2) UMBS_PREP_NC(2);
+    else if (nc == 4) UMBS_PREP_NC(4);
+    else if (nc == 8) UMBS_PREP_NC(8);
+    else UMBS_PREP_NC(16);
+#undef UMBS_PREP_NC
+#undef UMBS_PREP
     count_launches(1);
     return (int)cudaGetLastError();
 }

@@ -192,6 +192,86 @@ __global__ void add_norm_kernel(float* __restrict__ x, umbs_delta_t d, int has_d
     }
 }
 
+// The common case of add_norm_kernel in 16-byte pieces: one dense pending output, with or without a norm of its own, and an
+// RMS norm (or none) of the sum.  KEEP4 pieces per thread; the block's sums as fixed trees, one barrier each (every warp adds
+// up the warps' partial sums itself).
+__device__ __forceinline__ float block_sum_one_barrier(float v, float* red) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    v = warp_sum_pn(v);
+    if (lane == 0) red[warp] = v;
+    __syncthreads();
+    return warp_sum_pn(lane < nw ? red[lane] : 0.f);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
+template <typename T, int KEEP4>
+__global__ void add_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ post_w,
+                                    const int32_t* __restrict__ rows, const float* __restrict__ w, float w_offset, int width, float eps,
+                                    T* __restrict__ y, int64_t ldy, float* __restrict__ copy) {
+    __shared__ float red[2][32];
+    const int r = blockIdx.x, n4 = width / 4;
+    const int64_t src = rows ? rows[r] : r;
+    float4* xr = reinterpret_cast<float4*>(x + src * width);
+    const float4* dr = reinterpret_cast<const float4*>(delta + src * width);
+    float4 v[KEEP4], d[KEEP4];
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP4; ++i) {
+        const int e = threadIdx.x + i * blockDim.x;
+        v[i] = d[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (e < n4) { d[i] = dr[e]; v[i] = xr[e]; }
+        sum = fmaf(d[i].x, d[i].x, fmaf(d[i].y, d[i].y, fmaf(d[i].z, d[i].z, fmaf(d[i].w, d[i].w, sum))));
+    }
+    if (post_w != nullptr) {
+        const float inv = 1.f / sqrtf(block_sum_one_barrier(sum, red[0]) / (float)width + eps);
+#pragma unroll
+        for (int i = 0; i < KEEP4; ++i) {
+            const int e = threadIdx.x + i * blockDim.x;
+            if (e < n4) {
+                const float4 p = reinterpret_cast<const float4*>(post_w)[e];
+                d[i] = make_float4(d[i].x * inv * p.x, d[i].y * inv * p.y, d[i].z * inv * p.z, d[i].w * inv * p.w);
+            }
+        }
+    }
+    sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP4; ++i) {
+        v[i] = make_float4(v[i].x + d[i].x, v[i].y + d[i].y, v[i].z + d[i].z, v[i].w + d[i].w);
+        sum = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, sum))));
+    }
+    const float inv = w != nullptr ? 1.f / sqrtf(block_sum_one_barrier(sum, red[1]) / (float)width + eps) : 1.f;
+#pragma unroll
+    for (int i = 0; i < KEEP4; ++i) {
+        const int e = threadIdx.x + i * blockDim.x;
+        if (e >= n4) continue;
+        if (rows == nullptr) xr[e] = v[i];
+        if (copy != nullptr) reinterpret_cast<float4*>(copy + (int64_t)r * width)[e] = v[i];
+        if (y != nullptr) {
+            float4 o = v[i];
+            if (w != nullptr) {
+                const float4 g = reinterpret_cast<const float4*>(w)[e];
+                o = make_float4(o.x * inv * (w_offset + g.x), o.y * inv * (w_offset + g.y), o.z * inv * (w_offset + g.z), o.w * inv * (w_offset + g.w));
+            }
+            store4(y + (int64_t)r * ldy + 4 * e, o);
+        }
+    }
+}
+
+template <typename T>
+static void launch_add_norm_vec(float* x, const umbs_delta_t& d, const int32_t* rows, int n, const float* w, float w_offset, int width,
+                                float eps, T* y, int64_t ldy, float* copy, cudaStream_t st) {
+    // few rows: spread each over as many threads as there are pieces; many: four pieces per thread
+    const int n4 = width / 4, keep = n <= 148 ? (n4 <= 1024 ? 1 : 2) : 4;
+    const int threads = ((n4 + keep - 1) / keep + 31) / 32 * 32;
+    if (keep == 1) add_norm_vec_kernel<T, 1><<<n, threads, 0, st>>>(x, d.delta, d.norm_w, rows, w, w_offset, width, eps, y, ldy, copy);
+    else if (keep == 2) add_norm_vec_kernel<T, 2><<<n, threads, 0, st>>>(x, d.delta, d.norm_w, rows, w, w_offset, width, eps, y, ldy, copy);
+    else add_norm_vec_kernel<T, 4><<<n, threads, 0, st>>>(x, d.delta, d.norm_w, rows, w, w_offset, width, eps, y, ldy, copy);
+}
+
 // One block per token: the embedding row through an RMS norm, in fp32 and (for a product that reads it) as T.
 template <typename T>
 __global__ void embedding_norm_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float scale, const float* __restrict__ w,
@@ -410,8 +490,13 @@ static int add_norm_run(int dtype, float* x, const umbs_delta_t* d, const int32_
     umbs_delta_t dd{};
     if (d != nullptr) dd = *d;
     if (dd.delta_mult == 0.f && dd.delta2 == nullptr) dd.delta_mult = 1.f;
-    UMBS_DISPATCH_T(dtype, add_norm_kernel<T><<<n, threads, 0, st>>>(x, dd, d != nullptr, rows, kind, w, b, w_offset, alpha, width,
-                                                                     eps, (T*)y, ldy, copy));
+    const uintptr_t ptrs = (uintptr_t)x | (uintptr_t)dd.delta | (uintptr_t)dd.norm_w | (uintptr_t)w | (uintptr_t)copy | (uintptr_t)y;
+    if (d != nullptr && dd.delta != nullptr && dd.pair_out == nullptr && dd.shared == nullptr && dd.delta2 == nullptr && dd.scale == nullptr &&
+        dd.mult == 1.f && dd.delta_mult == 1.f && (kind == UMBS_NORM_RMS || kind == kNormNone) && width % 4 == 0 && ldy % 4 == 0 && ptrs % 16 == 0)
+        UMBS_DISPATCH_T(dtype, launch_add_norm_vec<T>(x, dd, rows, n, kind == kNormNone ? nullptr : w, w_offset, width, eps, (T*)y, ldy, copy, st));
+    else
+        UMBS_DISPATCH_T(dtype, add_norm_kernel<T><<<n, threads, 0, st>>>(x, dd, d != nullptr, rows, kind, w, b, w_offset, alpha, width,
+                                                                         eps, (T*)y, ldy, copy));
     count_launches(1);
     return (int)cudaGetLastError();
 }

@@ -461,3 +461,77 @@ def moe_route_scaled(h, w_router, top: int, mode: int, weight_scale: float = 1.0
                                            _p(sel_w), _p(grp_off), _p(pair_tok), _p(pair_pos), _p(scratch), None, None,
                                            _stream()), "moe_route_scaled")
     return sel_w, grp_off, pair_tok, pair_pos, scratch[2 * E:].view(n, top)
+
+
+# ---------------------------------------------------------------------------------------------- norms behind blocks, rank-one memories
+def add_post_norm(x, delta, post_w, w, eps: float, dtype=torch.float32, rows=None, want_copy: bool = False):
+    """x [n, width] fp32 += delta / rms(delta) * post_w (in place when ``rows`` is None), then x / rms(x) * w as ``dtype``."""
+    n = x.shape[0] if rows is None else rows.numel()
+    y = torch.empty((n, x.shape[1]), dtype=dtype, device=x.device)
+    copy = torch.empty((n, x.shape[1]), dtype=torch.float32, device=x.device) if want_copy else None
+    d = S.Delta()
+    d.delta, d.mult, d.delta_mult, d.norm_w = delta.data_ptr(), 1.0, 1.0, post_w.data_ptr()
+    S.check(S.load().umbs_add_norm_ex(_mode(y), _p(x), C.byref(d), _p(rows), n, S.UMBS_NORM_RMS, _p(w), None, 0.0, 1.0, x.shape[1],
+                                      float(eps), _p(y), _p(copy), _stream()), "add_norm_ex")
+    return (y, copy) if want_copy else y
+
+
+def add_rows(x, out, delta=None, post_w=None, eps: float = 0.0):
+    """x [n, width] fp32 += delta (through an RMS norm with ``post_w`` if given); out[:, :width] = x in out's dtype (out may have
+    a longer row)."""
+    d = None
+    if delta is not None:
+        d = S.Delta()
+        d.delta, d.mult, d.delta_mult, d.norm_w = delta.data_ptr(), 1.0, 1.0, post_w.data_ptr() if post_w is not None else None
+    S.check(S.load().umbs_add_rows(_mode(out), _p(x), C.byref(d) if d is not None else None, x.shape[0], x.shape[1], float(eps), _p(out),
+                                   out.stride(0), None, _stream()), "add_rows")
+    return out
+
+
+def embedding_norm(ids, table, w, eps: float, scale: float = 1.0, copy=None):
+    """fp32 [n, width]: RMS norm (weight w) of the rows table[ids] * scale; ``copy``: a second place for them, in the table's dtype."""
+    y = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    S.check(S.load().umbs_embedding_norm(_mode(table), _p(ids), _p(table), float(scale), _p(w), float(eps), _p(y), _p(copy),
+                                         copy.stride(0) if copy is not None else 0, ids.numel(), table.shape[1], _stream()), "embedding_norm")
+    return y
+
+
+def memory_layout(kind: str, heads, kv_heads, dim, vdim, taps, conv_w, conv_state, decay_rate, dt_bias, state, conv_b=None, skip=None):
+    """umbs_memory_t of a "gated_delta" layer (projection q | k | v | gate | strength | decay input) or an "ssd" layer (gate | v | k
+    | q | step size) and the columns where the projection's gate begins."""
+    gd, hv = kv_heads * dim, heads * vdim
+    delta = kind == "gated_delta"
+    m = S.Memory()
+    m.rule, m.unit = (S.UMBS_MEMORY_DELTA, 1) if delta else (S.UMBS_MEMORY_ADD, 0)
+    m.heads, m.kv_heads, m.dim, m.vdim, m.taps = heads, kv_heads, dim, vdim, taps
+    m.off_conv, m.off_q, m.off_k, m.off_v = (0, 0, gd, 2 * gd) if delta else (hv, hv + gd, hv, 0)
+    m.off_strength, m.off_decay = (2 * gd + 2 * hv, 2 * gd + 2 * hv + heads) if delta else (-1, 2 * gd + 2 * hv)
+    for name, t in (("conv_w", conv_w), ("conv_b", conv_b), ("conv_state", conv_state), ("decay_rate", decay_rate), ("dt_bias", dt_bias),
+                    ("skip", skip), ("state", state)):
+        setattr(m, name, t.data_ptr() if t is not None else None)
+    return m, 2 * gd + hv if delta else 0
+
+
+def memory_prep(proj, mem, batch: RaggedBatch, slots: int):
+    """proj fp32 [T, .] -> (qkv [T, channels rounded up to 4], gates [T, heads, 2] (log decay, strength), kq [T, kv_heads]), fp32."""
+    T, ch = proj.shape[0], 2 * mem.kv_heads * mem.dim + mem.heads * mem.vdim
+    f = dict(dtype=torch.float32, device=proj.device)
+    qkv, gates, kq = torch.empty((T, (ch + 3) // 4 * 4), **f), torch.empty((T, mem.heads, 2), **f), torch.empty((T, mem.kv_heads), **f)
+    S.check(S.load().umbs_memory_prep(_p(proj), proj.stride(0), C.byref(mem), C.byref(batch.c), slots, _p(qkv), qkv.stride(0), _p(gates),
+                                      _p(kq), _stream()), "memory_prep")
+    return qkv, gates, kq
+
+
+def memory_run(qkv, gates, kq, mem, batch: RaggedBatch):
+    o = torch.empty((qkv.shape[0], mem.heads * mem.vdim), dtype=torch.float32, device=qkv.device)
+    S.check(S.load().umbs_memory_run(_p(qkv), qkv.stride(0), _p(gates), _p(kq), C.byref(mem), C.byref(batch.c), _p(o), _stream()),
+            "memory_run")
+    return o
+
+
+def gated_norm(o, gate, parts: int, w, gate_first: bool, eps: float, dtype=torch.float32):
+    """unit(o silu(gate)) * w (``gate_first``) or unit(o) * w * silu(gate), unit RMS over each of ``parts`` equal parts of a row."""
+    out = torch.empty(o.shape, dtype=dtype, device=o.device)
+    S.check(S.load().umbs_gated_norm(_mode(out), _p(o), _p(gate), gate.stride(0), o.shape[0], o.shape[1], parts, _p(w), w.numel(),
+                                     int(gate_first), float(eps), _p(out), _stream()), "gated_norm")
+    return out

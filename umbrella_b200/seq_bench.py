@@ -813,3 +813,188 @@ def run_subivik(args):
                        "l2": "whole-model runs stream more than L2 per step; kernel table flushes L2 between runs"},
             "sizes": sizes, "kernels": table}
     print(json.dumps(line))
+
+
+# ---------------------------------------------------------------------------------------------- the Ralapel family
+def ralapel_config(width: int, layers: int = 8) -> dict:
+    """A Ralapel config with the layer sizes of a model of this width: state-space layers (heads of 64 over the width, 128 state
+    dimensions, one group), gated delta layers (heads of 128 over the width, half as many query / key heads), latent attention
+    as Kulisun's; dense feed-forward of 2 x width as Zedotar's.  ``layers`` layer runs: six layers with a span of two that
+    runs a second time, then the three kinds in turn."""
+    heads = max(2, width // 128)
+    ssd = dict(type="mamba2", mixer=dict(heads=width // 64, vdim=64, state=128, groups=1, norm_groups=1, conv=4))
+    dlt = dict(type="delta", mixer=dict(heads=heads, kv_heads=heads // 2, dim=128, vdim=128, conv=4))
+    lat = dict(type="latent_attention", mixer=dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=width // 4, scale=192 ** -0.5,
+                                                   rot=dict(base=1e6, dims=64)))
+    mlp = dict(kind="dense", ff=2 * width)
+    return dict(architecture="Ralapel", width=width, vocab=32768, norm=dict(eps=1e-6), loop=dict(start=1, stop=3, times=2),
+                layers=[dict((ssd, dlt, lat)[i % 3], mlp=mlp) for i in range(layers - 2)])
+
+
+def bench_ralapel(width, layers, device, prompt, ctx, batches, timer):
+    from .models.ralapel import Ralapel, spec_from_config
+    spec = spec_from_config(ralapel_config(width, layers))
+    m = Ralapel(spec, device=device, dtype=torch.bfloat16, slots=max(batches), max_tokens=prompt + ctx)
+    return bench_seq_model(m, spec, prompt, ctx, batches, timer)
+
+
+def kernel_table_ralapel(am, zm, km, device, timer, T=4096):
+    """Device time of each Ralapel mechanism at prefill size (one sequence of T tokens) and at decode size (8 and 64 sequences
+    behind 512 tokens), with its roofline fractions, and the like kernels of the Zedotar and (latent attention) Kulisun paths
+    measured the same way in the same run (``like`` names the pairing)."""
+    from . import _lib_seq as S, ops_seq as Q
+    hbm, tflops, how = _peaks()
+    sp, W = am.spec, am.spec.width
+    fp32_peak = 148 * 128 * 2 * 1.965e-3
+    rows = []
+
+    def add(name, ms, nbytes=0, flops=0, like=None, flops32=0):
+        r = dict(kernel=name, ms=round(ms, 4))
+        if flops32:
+            r["fp32_tflops"], r["frac_of_fp32_fma_peak"] = round(flops32 / ms / 1e9, 2), round(flops32 / ms / 1e9 / fp32_peak, 3)
+        if flops:
+            r["tflops"], r["frac_of_bf16_peak"] = round(flops / ms / 1e9, 1), round(flops / ms / 1e9 / tflops, 3)
+        if nbytes:
+            r["gb_s"], r["frac_of_hbm_peak"] = round(nbytes / ms / 1e6, 1), round(nbytes / ms / 1e6 / hbm, 3)
+        if like:
+            r["like"] = like
+        rows.append(r)
+    pick = lambda spec, kind: next(i for i, l in enumerate(spec.layers) if l.mixer == kind)
+    ai = pick(sp, "latent_attention")
+    zsp, ksp = zm.spec, km.spec
+    zi = pick(zsp, "mlstm")
+    mls, mw, lat, aw, kw = zsp.layers[zi], zm.weights[zi], sp.layers[ai], am.weights[ai], km.weights[0]
+    klat = ksp.layers[0]
+    bf = dict(dtype=torch.bfloat16, device=device)
+    ctx = 512
+    for m in (am, zm, km):
+        m.cache.reserve_length(T)
+    loop_in = am.head_weights["loop_in"]
+    for n, tag in ((T, f"prefill T={T}"), (8, "decode T=8"), (64, "decode T=64")):
+        nseq = 1 if n == T else n
+        per = n // nseq
+        pos0 = 0 if n == T else ctx
+        batch = Q.RaggedBatch([(s, per, pos0, 0) for s in range(nseq)], device)
+        x, d = torch.randn(n, W, device=device), torch.randn(n, W, device=device)
+        h, cat = torch.randn(n, W, **bf), torch.randn(n, 2 * W, **bf)
+        # norms
+        ms = timer(lambda: Q.add_post_norm(x, d, aw["post_norm"], aw["norm"], sp.norm_eps, torch.bfloat16))
+        add(f"norm behind the block + residual add + rms norm ({tag})", ms, nbytes=n * W * (4 + 4 + 4 + 2), like="residual add + rms norm")
+        ms = timer(lambda: Q.add_rms_norm(x, d, mw["norm"], 1.0, zsp.norm_eps, torch.bfloat16))
+        add(f"zedotar residual add + rms norm ({tag})", ms, nbytes=n * W * (4 + 4 + 4 + 2))
+        ms = timer(lambda: Q.add_rows(x, cat, d, aw["post_norm"], sp.norm_eps))
+        add(f"norm behind the block + residual add + rows of a pass ({tag})", ms, nbytes=n * W * (4 + 4 + 4 + 2), like="residual add + rms norm")
+        # products
+        ms = timer(lambda: Q.gemm(cat, loop_in, out_f32=True))
+        add(f"gemm in front of a pass [{n} x {2 * W}] x [{W} x {2 * W}] ({tag})", ms, nbytes=loop_in.numel() * 2 + n * W * (4 + 4),
+            flops=4 * n * W * W, like="gemm in-projection")
+        win = mw["w_in"]
+        ms = timer(lambda: Q.gemm(h, win, out_f32=True))
+        add(f"zedotar gemm in-projection [{n} x {W}] x [{win.shape[0]} x {W}] ({tag})", ms,
+            nbytes=win.numel() * 2 + n * W * 2 + n * win.shape[0] * 4, flops=2 * n * W * win.shape[0])
+        gu = aw["s_gu"]
+        ms = timer(lambda: Q.gemm(h, gu, dual=S.UMBS_ACT_GELU_TANH))
+        add(f"gemm dense gate|up + gelu [{n} x {W}] x [{gu.shape[0]} x {W}] (the kernel Zedotar's layers run; {tag})", ms,
+            nbytes=gu.numel() * 2 + n * W * 2 + n * gu.shape[0], flops=2 * n * W * gu.shape[0])
+        # the memories beside mLSTM
+        for kind, name in (("gated_delta", "gated delta"), ("ssd", "state space")):
+            i = pick(sp, kind)
+            l, w, u = sp.layers[i], am.weights[i], sp.layers[i].state_index
+            H, G, D, V = l.heads, l.kv_heads, l.dim, l.vdim
+            proj = torch.randn(n, w["w_in"].shape[0], device=device)
+            mem, g0 = Q.memory_layout(kind, H, G, D, V, l.taps, w["conv_w"], am.cache.conv_state[u], w["decay_rate"], w["dt_bias"],
+                                      am.cache.mem_state[u], w.get("conv_b"), w.get("skip"))
+            gate, ch = proj[:, g0:], 2 * G * D + H * V
+            qkv, gates, kq = Q.memory_prep(proj, mem, batch, am.cache.slots)
+            o = Q.memory_run(qkv, gates, kq, mem, batch)
+            parts, first = (H, False) if kind == "gated_delta" else (l.norm_parts, True)
+            fl = (6 if kind == "gated_delta" else 4) * n * H * D * V
+
+            def all_three():
+                qkv, gates, kq = Q.memory_prep(proj, mem, batch, am.cache.slots)
+                return Q.gated_norm(Q.memory_run(qkv, gates, kq, mem, batch), gate, parts, w["out_norm"], first, sp.norm_eps, torch.bfloat16)
+            st = nseq * H * D * V * 8
+            shape = f"{H} heads of {D} x {V}, {G} query/key heads"
+            ms = timer(all_three)
+            add(f"{name}: convolution + gates + recurrence + gated norm, fp32, {shape} ({tag})", ms,
+                nbytes=n * (ch + H * V) * 4 + n * H * V * 2 + st, flops32=fl, like="zedotar mlstm")
+            ms = timer(lambda: Q.memory_prep(proj, mem, batch, am.cache.slots))
+            add(f"  {name}: convolution + silu + unit norms + gates ({tag})", ms, nbytes=n * (2 * ch + 4 * H) * 4, like="zedotar attention prep")
+            ms = timer(lambda: Q.memory_run(qkv, gates, kq, mem, batch))
+            add(f"  {name}: recurrence ({tag})", ms, nbytes=n * (ch + H * V) * 4 + st, flops32=fl, like="zedotar mlstm")
+            ms = timer(lambda: Q.gated_norm(o, gate, parts, w["out_norm"], first, sp.norm_eps, torch.bfloat16))
+            add(f"  {name}: gated norm ({tag})", ms, nbytes=n * H * V * (4 + 4 + 2), like="residual add + rms norm")
+        ld = 2 * mls.heads * (mls.dim + mls.vdim) + 2 * mls.heads
+        mproj = torch.randn(n, ld, device=device)
+        mstate = zm.cache.mlstm_state[zi]
+        ms = timer(lambda: Q.mlstm(mproj, mw["bias_in"], batch, mls.heads, mls.dim, mls.vdim, mls.gate_cap, zsp.norm_eps, mw["out_norm"],
+                                   mstate, torch.bfloat16))
+        add(f"zedotar mlstm: gates + recurrence + normaliser + unit norm + gate, fp32, {mls.heads} heads of {mls.dim} x {mls.vdim} ({tag})", ms,
+            nbytes=n * ld * 4 + n * mls.heads * mls.vdim * 2 + nseq * mls.heads * mls.dim * (mls.vdim + 1) * 8,
+            flops32=4 * n * mls.heads * mls.dim * (mls.vdim + 1))
+        zat = next(l for l in zsp.layers if l.taps > 1)
+        za = zm.weights[zsp.layers.index(zat)]
+        zh, zg, zd = zat.heads, zat.kv_heads, zat.dim
+        zpr = torch.randn(n, zh * zd + zg * zd + zh * zat.vdim, device=device)
+        zcs = zm.cache.conv_state[zsp.layers.index(zat)]
+        ms = timer(lambda: Q.attention_prep(zpr, za.get("bias_in"), batch, zh, zg, zd, zd, zat.rot_dims, za["inv_freq"], zat.rot_mag, True,
+                                            zat.taps, za["conv_w"], zcs, torch.bfloat16))
+        add(f"zedotar attention prep: convolution + rotary -> q, key|value rows ({tag})", ms, nbytes=n * (zh + zg) * zd * 4 + n * (zh + 2 * zg) * zd * 2)
+        # latent attention beside Kulisun's (the same kernels, sink and gate off)
+        for l, w, model, who, sink, gated in ((lat, aw, am, "", None, False), (klat, kw, km, "kulisun ", kw["sink"], True)):
+            H, D, Rt, R, V = l.heads, l.dim, l.rope_dim, l.kv_rank, l.vdim
+            KD = R + Rt
+            proj = torch.randn(n, H * (D + Rt) + KD + (H * V if gated else 0), device=device)
+            gate = proj[:, H * (D + Rt) + KD:] if gated else None
+            what = "sink, gate" if gated else "plain softmax"
+            ms = timer(lambda: Q.latent_prep(proj, batch, H, D, Rt, R, w["kv_norm"], 1e-6, l.rot_dims, w["inv_freq"], l.rot_mag, torch.bfloat16))
+            add(f"{who}latent norm + rotary ({tag})", ms, nbytes=n * (H * (D + Rt) + KD) * (4 + 2) + n * H * Rt * 4,
+                like=None if who else "kulisun latent norm + rotary")
+            keys = sum(p + 1 for p in range(pos0, pos0 + per)) * nseq
+            if n == T:
+                q, kvh, ks = torch.randn(n, H * (D + Rt), **bf), torch.randn(n, H * (D + V), **bf), torch.randn(n, KD, **bf)
+                ms = timer(lambda: Q.window_attention_shared(q, kvh[:, :H * D], ks[:, R:], kvh[:, H * D:], batch, H, l.scale, sink=sink,
+                                                             use_sink=gated, gate=gate))
+                add(f"{who}attention over per-head keys + shared rotated part, causal, {what}, fp32 scores ({tag})", ms,
+                    nbytes=n * (H * (D + Rt) + H * (D + V) + Rt + H * V) * 2 + (n * H * V * 4 if gated else 0),
+                    flops32=2 * keys * H * (D + Rt + V), like=None if who else "kulisun attention over per-head keys")
+            else:
+                ring = model.cache.ring[ai if not who else 0]
+                qa, c = torch.randn(n, H, KD, device=device), torch.randn(n, KD, **bf)
+                ms = timer(lambda: Q.latent_attention_shared(qa, c, ring, batch, H, R, Rt, l.scale, sink=sink, use_sink=gated, append=False))
+                add(f"{who}latent attention over [latent | shared part] keys, causal, {what}, fp32 scores ({tag})", ms,
+                    nbytes=n * H * (KD * 4 + R * 2) + keys * KD * 2, flops32=2 * keys * H * (KD + R),
+                    like=None if who else "kulisun latent attention")
+    return rows, how
+
+
+def run_ralapel(args):
+    from . import _lib_seq
+    device = "cuda:0"
+    timer = Timer(device)
+    hbm, tflops, how = _peaks()
+    sizes, table = [], None
+    launches0 = _lib_seq.load().umbs_launch_count()
+    for width in (1024, 2048):
+        layers, prompt, ctx = 8, 2048, 512
+        am, a = bench_ralapel(width, layers, device, prompt, ctx, (1, 8, 64), timer)
+        zm, z = bench_zedotar(width, layers, device, prompt, ctx, (1, 8, 64), timer)
+        km, k = bench_kulisun(width, layers, device, prompt, ctx, (1, 8, 64), timer)
+        rounded = lambda r: {n: round(v, 3) for n, v in r.items()}
+        sizes.append({"width": width, "layer_runs": layers, "ralapel_bf16": rounded(a), "zedotar_bf16": rounded(z), "kulisun_bf16": rounded(k)})
+        if width == 2048:
+            table, _ = kernel_table_ralapel(am, zm, km, device, timer)
+        del am, zm, km
+        torch.cuda.empty_cache()
+    launches = _lib_seq.load().umbs_launch_count() - launches0
+    head = sizes[-1]["ralapel_bf16"]
+    line = {"metric": "decode tokens/sec at batch 64 (Ralapel bf16, width 2048, 8 layer runs, synthetic weights)",
+            "value": head["decode_b64_tok_s"], "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16",
+            "data": "synthetic", "vs_baseline": None, "gpu_launches": int(launches),
+            "config": {"name": "ralapel", "workload": "prefill 1 x 2048 and 4 x 2048 tokens; decode at batch 1 / 8 / 64 behind a "
+                       "512-token context; Zedotar bf16 (the closest family: matrix memories, attention, gelu-gated dense feed-forward) and "
+                       "Kulisun bf16 (latent attention in every layer) of the same width and depth beside it",
+                       "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": how},
+                       "l2": "whole-model runs stream more than L2 per step; kernel table flushes L2 between runs"},
+            "sizes": sizes, "kernels": table}
+    print(json.dumps(line))
