@@ -288,3 +288,63 @@ def test_state_cache_of_subivik_layers():
     assert c.tm_state[6].shape == (2, 3, 20, 20) and c.shift[6].shape == (2, 2, 80) and c.shift[1] is None
     c.reserve_length(70)
     assert c.capacity == 128 and c.kv_cache[0].shape[1] == 24 and c.kv_cache[1].shape[1] == 128 and c.kv_cache[4].shape[1] == 128
+
+
+# ---------------------------------------------------------------------------------------------- the Ralapel family
+def test_ralapel_config_reader_and_tensor_names():
+    import copy
+    import ral_helpers as U
+    from umbrella_b200.models.ralapel import layer_tensor_names, spec_from_config, synth_tensors
+    spec = spec_from_config(U.MIXED)
+    assert (spec.width, spec.vocab, spec.norm_eps, spec.norm_kind, spec.embed_norm, spec.loop) == (72, 101, 1e-5, "rms", True, (1, 4, 3))
+    assert all(l.form == "prenorm" and l.post_norm and not l.shift and not l.depth_average and l.norm_kind == "rms" for l in spec.layers)
+    d, m, a, m2, a2, d2 = spec.layers
+    assert (d.mixer, d.heads, d.kv_heads, d.dim, d.vdim, d.taps, d.mlp.shared_ff, d.mlp.act) == ("gated_delta", 6, 3, 12, 20, 3, 40, "gelu_tanh")
+    assert (m.mixer, m.heads, m.vdim, m.dim, m.kv_heads, m.norm_parts, m.taps, m.mlp) == ("ssd", 4, 10, 14, 2, 5, 4, None)
+    assert (a.mixer, a.heads, a.dim, a.rope_dim, a.vdim, a.kv_rank, a.rot_dims, a.rot_base, a.rot_pairs, a.q_rank, a.window) == \
+        ("latent_attention", 3, 10, 6, 14, 20, 6, 300.0, "neighbours", 0, 0)
+    assert (a.attn_mode, a.gate_kind, a.learned_sink, a.scale) == ("softmax", 0, False, U.MIXED["layers"][2]["mixer"]["scale"])
+    assert (m2.taps, m2.norm_parts, m2.kv_heads, d2.taps, d2.kv_heads, a2.rot_base) == (1, 1, 1, 2, 2, 1000.0)
+    assert [i for i, _ in spec.layer_runs()] == [0, 1, 2, 3, 1, 2, 3, 1, 2, 3, 4, 5]
+    assert [r for r, (_, b) in enumerate(spec.layer_runs()) if b] == [1, 4, 7]
+    names = {n for i in range(len(spec.layers)) for v in layer_tensor_names(spec, i).values() for n in ([v] if isinstance(v, str) else v)}
+    top = {"embed", "embed.norm", "head", "final.norm"}
+    tensors = U.random_tensors(U.MIXED)
+    assert names | top | {"loop.in"} == set(tensors)
+    assert {k: tuple(v.shape) for k, v in synth_tensors(spec, 1).items()} == {k: tuple(v.shape) for k, v in tensors.items()}
+    plain = spec_from_config({k: v for k, v in U.PLAIN.items() if k != "loop"})
+    assert plain.loop is None and plain.layer_runs() == [(0, False), (1, False), (2, False)]
+    assert "loop.in" not in synth_tensors(plain, 1)
+    for path, value in ((("layers", 1, "mixer", "norm_groups"), 7), (("layers", 0, "mixer", "kv_heads"), 4), (("layers", 1, "mixer", "groups"), 3),
+                        (("layers", 2, "mixer", "rot", "dims"), 8), (("layers", 2, "type"), "attention"), (("architecture",), "Zedotar")):
+        bad = copy.deepcopy(U.MIXED)
+        at = bad
+        for k in path[:-1]:
+            at = at[k]
+        at[path[-1]] = value
+        with pytest.raises(ValueError):
+            spec_from_config(bad)
+
+
+def test_state_cache_of_looped_memories():
+    import ral_helpers as U
+    from umbrella_b200.attn.state_cache import SequenceStateCache
+    from umbrella_b200.models.ralapel import spec_from_config
+    from umbrella_b200.models.seq_model import SeqStateModel
+    spec = spec_from_config(U.MIXED)
+    c = SequenceStateCache(spec, slots=2, device="cpu", dtype=torch.float32, capacity=24)
+    assert len(c.units) == 12 and [l.state_index for l in spec.layers] == [0, 1, 2, 3, 10, 11]
+    assert c.mem_state[0].shape == (2, 6, 20, 12) and c.conv_state[0].shape == (2, 2, 2, 2 * 36 + 120)
+    for r in (1, 4, 7):                                               # every pass has a state, a cache and convolution rows of its own
+        assert c.mem_state[r].shape == (2, 4, 10, 14) and c.conv_state[r].shape == (2, 2, 3, 40 + 56)
+        assert c.ring[r + 1].shape == (2, 24, 26) and c.mem_state[r + 2].shape == (2, 2, 24, 33) and c.conv_state[r + 2] is None
+    assert len({c.mem_state[r].data_ptr() for r in (1, 4, 7)}) == 3
+    c.mem_state[4][1].fill_(2.0), c.conv_state[4][1, 1].fill_(3.0), c.ring[5][1, 23].fill_(4.0)
+    c.reserve_length(30)
+    s = [c.alloc_slot() for _ in range(3)]
+    assert c.capacity == 48 and c.slots == 4 and c.ring[5].shape == (4, 48, 26) and len(set(s)) == 3
+    assert float(c.mem_state[4][1].min()) == 2.0 and float(c.conv_state[4][1, 1].min()) == 3.0 and float(c.ring[5][1, 23].min()) == 4.0
+    assert c.state_bytes_per_slot() > 0
+    spec.loop = (2, 2, 1)
+    with pytest.raises(ValueError):
+        SeqStateModel(spec, device="cpu")

@@ -194,6 +194,29 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src));
 }
 
+// Two fp32 numbers in one 64-bit register and the packed multiply-add on them (each half rounds as its scalar form does).
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
 // RL lanes share a value column and hold RPL of its rows each (rows 4 (r + RL i) .. + 3 of lane r, so that the 16-byte loads
 // of the lanes that share a column are consecutive); a lane holds CPL columns.  The whole state slice stays in registers for
 // the step.  Tokens run in order; TB at a time are staged (q, k, the block's value columns, decay, strength, k . q) in a ring
@@ -217,7 +240,7 @@ __global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __r
     const int hv = m.heads * V, ncol = min(CT, V - c0);
     const float skip = m.skip != nullptr ? m.skip[h] : 0.f;
     float* st = m.state + ((int64_t)slot * m.heads + h) * V * D;                   // S[column][row]
-    float S[CPL][RPL];
+    f32x2 S[CPL][RPL / 2];                                                         // neighbouring rows in pairs
     int col[CPL];
 #pragma unroll
     for (int c = 0; c < CPL; ++c) {
@@ -227,13 +250,15 @@ __global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __r
 #pragma unroll
         for (int i = 0; i < RPL / 4; ++i) {
             const int r = 4 * (rl + RL * i);
+            float f[4];
             if (have && D % 4 == 0) {
-                const float4 f = r < D ? *reinterpret_cast<const float4*>(sc + r) : make_float4(0.f, 0.f, 0.f, 0.f);
-                S[c][4 * i] = f.x; S[c][4 * i + 1] = f.y; S[c][4 * i + 2] = f.z; S[c][4 * i + 3] = f.w;
+                *reinterpret_cast<float4*>(f) = r < D ? *reinterpret_cast<const float4*>(sc + r) : make_float4(0.f, 0.f, 0.f, 0.f);
             } else {
 #pragma unroll
-                for (int x = 0; x < 4; ++x) S[c][4 * i + x] = (have && r + x < D) ? sc[r + x] : 0.f;
+                for (int x = 0; x < 4; ++x) f[x] = (have && r + x < D) ? sc[r + x] : 0.f;
             }
+            S[c][2 * i] = pack2(f[0], f[1]);
+            S[c][2 * i + 1] = pack2(f[2], f[3]);
         }
     }
     // rows beyond dim and columns beyond vdim of every stage stay zero
@@ -298,42 +323,49 @@ __global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __r
         if (tid < nt) sg[4 * tid] = expf(sg[4 * tid]);                             // (the thread that copied it)
         __syncthreads();
         // the operands of a token are in registers before the token in front of it is worked on
-        struct Operands { float k[RPL], q[RPL], v[CPL]; float4 g; } op[2];
+        struct Operands { f32x2 k[RPL / 2], q[RPL / 2]; float v[CPL]; float4 g; } op[2];
         auto load = [&](Operands& x, int tt) {
             x.g = *reinterpret_cast<const float4*>(sg + 4 * tt);
 #pragma unroll
             for (int i = 0; i < RPL / 4; ++i) {
-                const float4 k4 = *reinterpret_cast<const float4*>(sk + tt * DP + 4 * (rl + RL * i));
-                const float4 q4 = *reinterpret_cast<const float4*>(sq + tt * DP + 4 * (rl + RL * i));
-                x.k[4 * i] = k4.x; x.k[4 * i + 1] = k4.y; x.k[4 * i + 2] = k4.z; x.k[4 * i + 3] = k4.w;
-                x.q[4 * i] = q4.x; x.q[4 * i + 1] = q4.y; x.q[4 * i + 2] = q4.z; x.q[4 * i + 3] = q4.w;
+                const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(sk + tt * DP + 4 * (rl + RL * i));
+                const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(sq + tt * DP + 4 * (rl + RL * i));
+                x.k[2 * i] = k4.x; x.k[2 * i + 1] = k4.y;
+                x.q[2 * i] = q4.x; x.q[2 * i + 1] = q4.y;
             }
 #pragma unroll
             for (int c = 0; c < CPL; ++c) x.v[c] = sv[tt * CT + col[c]];
         };
         auto walk = [&](const Operands& x, int tt) {
             const float dec = x.g.x, str = x.g.y, dot = x.g.z;
+            const f32x2 dec2 = pack2(dec, dec);
+            float dq[CPL], dk[CPL];
 #pragma unroll
             for (int c = 0; c < CPL; ++c) {
-                float aq[4] = {0.f, 0.f, 0.f, 0.f}, ak[4] = {0.f, 0.f, 0.f, 0.f};
+                f32x2 aq[2] = {0ull, 0ull}, ak[2] = {0ull, 0ull};
 #pragma unroll
-                for (int i = 0; i < RPL; i += 4)
-#pragma unroll
-                    for (int y = 0; y < 4; ++y) {
-                        if (DELTA) ak[y] = fmaf(S[c][i + y], x.k[i + y], ak[y]);
-                        aq[y] = fmaf(S[c][i + y], x.q[i + y], aq[y]);
-                    }
-                float dq = (aq[0] + aq[1]) + (aq[2] + aq[3]);
-                float dk = (ak[0] + ak[1]) + (ak[2] + ak[3]);
-#pragma unroll
-                for (int w = RL / 2; w > 0; w >>= 1) {
-                    if (DELTA) dk += __shfl_xor_sync(0xffffffffu, dk, w);
-                    dq += __shfl_xor_sync(0xffffffffu, dq, w);
+                for (int i = 0; i < RPL / 2; ++i) {
+                    if (DELTA) ak[i & 1] = fma2(S[c][i], x.k[i], ak[i & 1]);
+                    aq[i & 1] = fma2(S[c][i], x.q[i], aq[i & 1]);
                 }
-                const float u = DELTA ? str * fmaf(-dec, dk, x.v[c]) : str * x.v[c];
+                const float2 q0 = unpack2(aq[0]), q1 = unpack2(aq[1]), k0 = unpack2(ak[0]), k1 = unpack2(ak[1]);
+                dq[c] = (q0.x + q0.y) + (q1.x + q1.y);
+                dk[c] = (k0.x + k0.y) + (k1.x + k1.y);
+            }
 #pragma unroll
-                for (int i = 0; i < RPL; ++i) S[c][i] = fmaf(dec, S[c][i], x.k[i] * u);
-                if (rl == 0) so[tt * CT + col[c]] = fmaf(skip, x.v[c], fmaf(dot, u, dec * dq));
+            for (int w = RL / 2; w > 0; w >>= 1)
+#pragma unroll
+                for (int c = 0; c < CPL; ++c) {
+                    if (DELTA) dk[c] += __shfl_xor_sync(0xffffffffu, dk[c], w);
+                    dq[c] += __shfl_xor_sync(0xffffffffu, dq[c], w);
+                }
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) {
+                const float u = DELTA ? str * fmaf(-dec, dk[c], x.v[c]) : str * x.v[c];
+                const f32x2 u2 = pack2(u, u);
+#pragma unroll
+                for (int i = 0; i < RPL / 2; ++i) S[c][i] = fma2(dec2, S[c][i], mul2(x.k[i], u2));
+                if (rl == 0) so[tt * CT + col[c]] = fmaf(skip, x.v[c], fmaf(dot, u, dec * dq[c]));
             }
         };
         load(op[0], 0);
@@ -357,12 +389,14 @@ __global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __r
 #pragma unroll
         for (int i = 0; i < RPL / 4; ++i) {
             const int r = 4 * (rl + RL * i);
+            const float2 lo = unpack2(S[c][2 * i]), hi = unpack2(S[c][2 * i + 1]);
+            const float f[4] = {lo.x, lo.y, hi.x, hi.y};
             if (D % 4 == 0) {
-                if (r < D) *reinterpret_cast<float4*>(sc + r) = make_float4(S[c][4 * i], S[c][4 * i + 1], S[c][4 * i + 2], S[c][4 * i + 3]);
+                if (r < D) *reinterpret_cast<float4*>(sc + r) = make_float4(f[0], f[1], f[2], f[3]);
             } else {
 #pragma unroll
                 for (int x = 0; x < 4; ++x)
-                    if (r + x < D) sc[r + x] = S[c][4 * i + x];
+                    if (r + x < D) sc[r + x] = f[x];
             }
         }
     }
@@ -411,6 +445,75 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const float* __re
     const float inv = 1.f / sqrtf(ss / (float)size + eps);
     for (int e = me; e < size; e += step)
         out[(int64_t)t * width + e0 + e] = from_f32<T>(orow[e] * silu_mem(grow[e]) * inv * w[(e0 + e) % w_len]);
+}
+
+// The same in 16-byte pieces, a part's values held in registers (up to four pieces per lane of the warp, or per thread of the
+// block, that a part has).
+template <typename T>
+__global__ void gated_norm_vec_kernel(const float* __restrict__ o, const float* __restrict__ gate, int64_t ldg, int n_parts, int width, int parts,
+                                      const float* __restrict__ w, int w_len, int gate_first, float eps, int whole_block, T* __restrict__ out) {
+    __shared__ float red[32];
+    constexpr int KEEP4 = 4;
+    const int nw = blockDim.x >> 5, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int p = whole_block ? blockIdx.x : blockIdx.x * nw + warp;
+    const int me = whole_block ? threadIdx.x : lane, step = whole_block ? blockDim.x : 32;
+    if (p >= n_parts) return;                       // (never a part of a block that meets the barrier below)
+    const int t = p / parts, size = width / parts, e0 = (p - t * parts) * size, n4 = size / 4;
+    const float4* orow = reinterpret_cast<const float4*>(o + (int64_t)t * width + e0);
+    const float4* grow = reinterpret_cast<const float4*>(gate + (int64_t)t * ldg + e0);
+    float4 y[KEEP4], g[KEEP4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP4; ++i) {
+        const int e = me + i * step;
+        y[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (e < n4) { y[i] = orow[e]; g[i] = grow[e]; }
+    }
+#pragma unroll
+    for (int i = 0; i < KEEP4; ++i) {
+        g[i] = make_float4(silu_mem(g[i].x), silu_mem(g[i].y), silu_mem(g[i].z), silu_mem(g[i].w));
+        const float4 v = make_float4(y[i].x * g[i].x, y[i].y * g[i].y, y[i].z * g[i].z, y[i].w * g[i].w);
+        const float4 q = gate_first ? v : y[i];
+        ss = fmaf(q.x, q.x, fmaf(q.y, q.y, fmaf(q.z, q.z, fmaf(q.w, q.w, ss))));
+        y[i] = v;
+    }
+    ss = warp_sum_mem(ss);
+    if (whole_block) {
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        ss = warp_sum_mem(lane < nw ? red[lane] : 0.f);
+    }
+    const float inv = 1.f / sqrtf(ss / (float)size + eps);
+#pragma unroll
+    for (int i = 0; i < KEEP4; ++i) {
+        const int e = me + i * step;
+        if (e >= n4) continue;
+        const float4 ww = *reinterpret_cast<const float4*>(w + (e0 + 4 * e) % w_len);
+        T* dst = out + (int64_t)t * width + e0 + 4 * e;
+        const float r[4] = {y[i].x * inv * ww.x, y[i].y * inv * ww.y, y[i].z * inv * ww.z, y[i].w * inv * ww.w};
+        if constexpr (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+        } else {
+            __nv_bfloat162 a = __floats2bfloat162_rn(r[0], r[1]), b = __floats2bfloat162_rn(r[2], r[3]);
+            *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+        }
+    }
+}
+
+template <typename T>
+static void launch_gated_norm(const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w, int w_len,
+                              int gate_first, float eps, T* out, cudaStream_t st) {
+    const int size = width / parts, n_parts = n * parts;
+    const uintptr_t ptrs = (uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out;
+    if (size % 4 == 0 && ldg % 4 == 0 && w_len % 4 == 0 && ptrs % 16 == 0 && size <= 16384) {
+        const int block = size > 512, threads = block ? (size / 4 + 3) / 4 : 128;
+        gated_norm_vec_kernel<T><<<block ? n_parts : (n_parts + 3) / 4, (threads + 31) / 32 * 32, 0, st>>>(
+            o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
+    } else {
+        const int block = size > 256, threads = block ? (size >= 2048 ? 512 : 256) : 128;
+        gated_norm_kernel<T><<<block ? n_parts : (n_parts + 3) / 4, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len,
+                                                                                     gate_first, eps, block, out);
+    }
 }
 
 }  // namespace umbs
@@ -464,15 +567,18 @@ extern "C" int umbs_memory_run(const float* qkv, int64_t ld_qkv, const float* ga
     // 16-byte copies: every row, head and column tile must start on a 16-byte boundary
     const int vec = m->dim % 4 == 0 && m->vdim % 4 == 0 && ld_qkv % 4 == 0 && m->off_q % 4 == 0 && m->off_k % 4 == 0 && m->off_v % 4 == 0 &&
                     (uintptr_t)qkv % 16 == 0;
-#define UMBS_MEM(RL, RPL, TB)                                                                                                     \
-    (m->rule == UMBS_MEMORY_DELTA ? launch_memory<RL, RPL, 1, TB, true>(qkv, ld_qkv, gates, kq, *m, *batch, o, vec, st)            \
-                                  : launch_memory<RL, RPL, 1, TB, false>(qkv, ld_qkv, gates, kq, *m, *batch, o, vec, st))
+#define UMBS_MEM(RL, RPL, CPL, TB)                                                                                                     \
+    (m->rule == UMBS_MEMORY_DELTA ? launch_memory<RL, RPL, CPL, TB, true>(qkv, ld_qkv, gates, kq, *m, *batch, o, vec, st)            \
+                                  : launch_memory<RL, RPL, CPL, TB, false>(qkv, ld_qkv, gates, kq, *m, *batch, o, vec, st))
+    // few blocks (one long prompt): a column per lane, the shortest walk; many: two, so that a staged q and k serve both (the same
+    // additions in the same order either way)
+    const bool many = (int64_t)((m->vdim + 15) / 16) * m->heads * batch->n_seqs >= 4 * 148;
     int rc;
-    if (m->dim <= 32) rc = UMBS_MEM(8, 4, 16);
-    else if (m->dim <= 64) rc = UMBS_MEM(8, 8, 16);
-    else if (m->dim <= 128) rc = UMBS_MEM(8, 16, 16);
-    else if (m->dim <= 256) rc = UMBS_MEM(8, 32, 8);
-    else rc = UMBS_MEM(16, 32, 8);
+    if (m->dim <= 32) rc = many ? UMBS_MEM(8, 4, 2, 16) : UMBS_MEM(8, 4, 1, 16);
+    else if (m->dim <= 64) rc = many ? UMBS_MEM(8, 8, 2, 16) : UMBS_MEM(8, 8, 1, 16);
+    else if (m->dim <= 128) rc = many ? UMBS_MEM(8, 16, 2, 16) : UMBS_MEM(8, 16, 1, 16);
+    else if (m->dim <= 256) rc = UMBS_MEM(8, 32, 1, 8);
+    else rc = UMBS_MEM(16, 32, 1, 8);
 #undef UMBS_MEM
     if (rc) return rc;
     count_launches(1);
@@ -484,14 +590,8 @@ extern "C" int umbs_gated_norm(int dtype, const float* o, const float* gate, int
     if (n <= 0) return 0;
     if (o == nullptr || gate == nullptr || w == nullptr || out == nullptr || parts < 1 || width % parts != 0 || w_len < 1) return UMB_ERR_ARG;
     cudaStream_t st = (cudaStream_t)stream;
-    const int size = width / parts, n_parts = n * parts, block = size > 256;
-    const int threads = block ? (size >= 2048 ? 512 : 256) : 128;
-    const unsigned grid = block ? n_parts : (n_parts + 3) / 4;
-    if (dtype == UMBS_BF16)
-        gated_norm_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block,
-                                                                   (__nv_bfloat16*)out);
-    else if (dtype == UMBS_F32)
-        gated_norm_kernel<float><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, (float*)out);
+    if (dtype == UMBS_BF16) launch_gated_norm(o, gate, ldg, n, width, parts, w, w_len, gate_first, eps, (__nv_bfloat16*)out, st);
+    else if (dtype == UMBS_F32) launch_gated_norm(o, gate, ldg, n, width, parts, w, w_len, gate_first, eps, (float*)out, st);
     else return UMB_ERR_ARG;
     count_launches(1);
     return (int)cudaGetLastError();
