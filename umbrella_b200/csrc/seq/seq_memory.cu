@@ -262,8 +262,10 @@ __global__ void __launch_bounds__(32 * kMemWarps) memory_kernel(const float* __r
         }
     }
     // rows beyond dim and columns beyond vdim of every stage stay zero
-    for (int i = tid; i < kMemStages * STAGE; i += 32 * kMemWarps) mem_sm[i] = 0.f;
-    __syncthreads();
+    if (D < DP || ncol < CT) {
+        for (int i = tid; i < kMemStages * STAGE; i += 32 * kMemWarps) mem_sm[i] = 0.f;
+        __syncthreads();
+    }
     constexpr int NT = 32 * kMemWarps, P4 = DP / 4, C4 = CT / 4;
     auto issue = [&](int g) {
         float* sq = mem_sm + (g % kMemStages) * STAGE;
@@ -447,13 +449,12 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const float* __re
         out[(int64_t)t * width + e0 + e] = from_f32<T>(orow[e] * silu_mem(grow[e]) * inv * w[(e0 + e) % w_len]);
 }
 
-// The same in 16-byte pieces, a part's values held in registers (up to four pieces per lane of the warp, or per thread of the
-// block, that a part has).
-template <typename T>
+// The same in 16-byte pieces, a part's values held in registers (KEEP4 pieces per lane of the warp, or per thread of the block, that a
+// part has).
+template <typename T, int KEEP4>
 __global__ void gated_norm_vec_kernel(const float* __restrict__ o, const float* __restrict__ gate, int64_t ldg, int n_parts, int width, int parts,
                                       const float* __restrict__ w, int w_len, int gate_first, float eps, int whole_block, T* __restrict__ out) {
     __shared__ float red[32];
-    constexpr int KEEP4 = 4;
     const int nw = blockDim.x >> 5, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int p = whole_block ? blockIdx.x : blockIdx.x * nw + warp;
     const int me = whole_block ? threadIdx.x : lane, step = whole_block ? blockDim.x : 32;
@@ -506,9 +507,11 @@ static void launch_gated_norm(const float* o, const float* gate, int64_t ldg, in
     const int size = width / parts, n_parts = n * parts;
     const uintptr_t ptrs = (uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out;
     if (size % 4 == 0 && ldg % 4 == 0 && w_len % 4 == 0 && ptrs % 16 == 0 && size <= 16384) {
-        const int block = size > 512, threads = block ? (size / 4 + 3) / 4 : 128;
-        gated_norm_vec_kernel<T><<<block ? n_parts : (n_parts + 3) / 4, (threads + 31) / 32 * 32, 0, st>>>(
-            o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
+        const int block = size > 512, threads = block ? ((size / 4 + 3) / 4 + 31) / 32 * 32 : 128;
+        const unsigned grid = block ? n_parts : (n_parts + 3) / 4;
+        if (size <= 128) gated_norm_vec_kernel<T, 1><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
+        else if (size <= 256) gated_norm_vec_kernel<T, 2><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
+        else gated_norm_vec_kernel<T, 4><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
     } else {
         const int block = size > 256, threads = block ? (size >= 2048 ? 512 : 256) : 128;
         gated_norm_kernel<T><<<block ? n_parts : (n_parts + 3) / 4, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len,
@@ -573,8 +576,14 @@ extern "C" int umbs_memory_run(const float* qkv, int64_t ld_qkv, const float* ga
     // few blocks (one long prompt): a column per lane, the shortest walk; many: two, so that a staged q and k serve both (the same
     // additions in the same order either way)
     const bool many = (int64_t)((m->vdim + 15) / 16) * m->heads * batch->n_seqs >= 4 * 148;
+    // decoding: nothing to stage ahead, small blocks of shared memory
+    const bool one = batch->max_seq_len == 1;
     int rc;
-    if (m->dim <= 32) rc = many ? UMBS_MEM(8, 4, 2, 16) : UMBS_MEM(8, 4, 1, 16);
+    if (one && m->dim <= 32) rc = UMBS_MEM(8, 4, 1, 2);
+    else if (one && m->dim <= 64) rc = UMBS_MEM(8, 8, 1, 2);
+    else if (one && m->dim <= 128) rc = UMBS_MEM(8, 16, 1, 2);
+    else if (one && m->dim <= 256) rc = UMBS_MEM(8, 32, 1, 2);
+    else if (m->dim <= 32) rc = many ? UMBS_MEM(8, 4, 2, 16) : UMBS_MEM(8, 4, 1, 16);
     else if (m->dim <= 64) rc = many ? UMBS_MEM(8, 8, 2, 16) : UMBS_MEM(8, 8, 1, 16);
     else if (m->dim <= 128) rc = many ? UMBS_MEM(8, 16, 2, 16) : UMBS_MEM(8, 16, 1, 16);
     else if (m->dim <= 256) rc = UMBS_MEM(8, 32, 1, 8);

@@ -887,11 +887,16 @@ def kernel_table_ralapel(am, zm, km, device, timer, T=4096):
         # products
         ms = timer(lambda: Q.gemm(cat, loop_in, out_f32=True))
         add(f"gemm in front of a pass [{n} x {2 * W}] x [{W} x {2 * W}] ({tag})", ms, nbytes=loop_in.numel() * 2 + n * W * (4 + 4),
-            flops=4 * n * W * W, like="gemm in-projection")
+            flops=4 * n * W * W, like="zedotar gemm dense down")
         win = mw["w_in"]
         ms = timer(lambda: Q.gemm(h, win, out_f32=True))
         add(f"zedotar gemm in-projection [{n} x {W}] x [{win.shape[0]} x {W}] ({tag})", ms,
             nbytes=win.numel() * 2 + n * W * 2 + n * win.shape[0] * 4, flops=2 * n * W * win.shape[0])
+        down = mw["s_down"]
+        hf = torch.randn(n, down.shape[1], **bf)
+        ms = timer(lambda: Q.gemm(hf, down, out_f32=True))
+        add(f"zedotar gemm dense down [{n} x {down.shape[1]}] x [{W} x {down.shape[1]}] ({tag})", ms,
+            nbytes=down.numel() * 2 + hf.numel() * 2 + n * W * 4, flops=2 * n * down.numel())
         gu = aw["s_gu"]
         ms = timer(lambda: Q.gemm(h, gu, dual=S.UMBS_ACT_GELU_TANH))
         add(f"gemm dense gate|up + gelu [{n} x {W}] x [{gu.shape[0]} x {W}] (the kernel Zedotar's layers run; {tag})", ms,
