@@ -63,6 +63,13 @@ typedef void* umbs_stream_t; /* cudaStream_t */
 /* Activation of a plain product (the `unary` argument of umbs_gemm_unary; 0 = none). */
 #define UMBS_UNARY_TANH 1            /* tanh(z) */
 #define UMBS_UNARY_XIELU 2           /* z > 0: p0 z^2 + z / 2; z <= 0: p1 (exp(z) - 1 - z) + z / 2 */
+#define UMBS_UNARY_RELU2 3           /* max(z, 0)^2 */
+#define UMBS_UNARY_SILU 4            /* z sigmoid(z) */
+#define UMBS_UNARY_SCALE 5           /* p0 z */
+
+/* Gate of a mixer's normed output (umbs_gated_norm_ex). */
+#define UMBS_GATE_SILU 0             /* times z sigmoid(z) */
+#define UMBS_GATE_SIGMOID 1          /* times sigmoid(z) */
 
 /* Norm of the pre-norm layer form. */
 #define UMBS_NORM_RMS 0              /* x / sqrt(mean(x^2) + eps) * (offset + w) */
@@ -75,6 +82,7 @@ typedef void* umbs_stream_t; /* cudaStream_t */
                                       * scores the sum of its two largest scores, only experts of the `keep` best groups are
                                       * eligible; the `top` largest eligible scores, divided by their sum (+ 1e-20) */
 #define UMBS_ROUTE_SOFTMAX_ALL 2     /* softmax over all experts; the `top` largest scores, as they are (not renormalised) */
+#define UMBS_ROUTE_TABLE 3           /* no router: a table gives every token id its `top` experts, each with weight 1 / top */
 
 /* What a rank-one memory writes (umbs_memory_t.rule): S <- decay S + k u^T with */
 #define UMBS_MEMORY_ADD 0            /* u = strength v */
@@ -82,8 +90,13 @@ typedef void* umbs_stream_t; /* cudaStream_t */
 
 /* How attention turns scores into weights. */
 #define UMBS_ATTN_SOFTMAX 0          /* p = exp(s) / sum exp(s) */
-#define UMBS_ATTN_SOFTMAX_SINK 1     /* p = exp(s) / (1 + sum exp(s)): a sink of score 0 without a value */
+#define UMBS_ATTN_SOFTMAX_SINK 1     /* p = exp(s) / (exp(sink) + sum exp(s)): a sink without a value, of score 0 or a number per head */
 #define UMBS_ATTN_SIGMOID 2          /* p = sigmoid(s + bias[head]), not normalised over keys */
+
+/* What a cached-attention layer does with its values (umbs_layer_t.v_mix). */
+#define UMBS_VMIX_NONE 0
+#define UMBS_VMIX_SOURCE 1           /* later layers of the step mix this layer's values into theirs */
+#define UMBS_VMIX_MIX 2              /* v <- (1 - lambda) v + lambda v_source */
 
 /* One step's ragged batch.  Token t of the step belongs to sequence tok_seq[t] (an index into the seq_* arrays)
  * and sits at absolute position tok_pos[t]; a sequence's tokens are contiguous: [seq_start, seq_start + seq_len).
@@ -125,6 +138,7 @@ typedef struct {
     int plain;                 /* the shared (dense) part has no gate rows: W_down unary(W_up h), ws_gu = [shared_ff, width] */
     int unary;                 /* UMBS_UNARY_* of a plain part, with its two numbers */
     float unary_p0, unary_p1;
+    const int32_t* route_table;/* UMBS_ROUTE_TABLE: [vocab, top] experts per token id, distinct within a row, each in [0, experts) */
 } umbs_mlp_t;
 
 typedef struct umbs_layer_s {
@@ -244,6 +258,22 @@ typedef struct umbs_layer_s {
     const float* skip_w;       /* fp32 [heads] or NULL: o += skip v */
     int norm_parts;            /* state space: equal parts of the output that are normed on their own */
     float* mem_state;          /* fp32 [slots, heads, vdim, dim]: key index last */
+    /* pre-norm form without the norms in front: norm_w == NULL (then norm2_w too) -- the blocks read the residual stream itself */
+    /* cached attention, further options */
+    const float* q_norm_all_w; /* fp32 [heads dim] or NULL: RMS norm over all of a token's query numbers at once, before the rotation */
+    const float* k_norm_all_w; /* fp32 [kv_heads dim] or NULL: the same for its keys */
+    int v_mix;                 /* UMBS_VMIX_*; every layer that mixes has the source's kv_heads vdim */
+    float v_lambda;            /* UMBS_VMIX_MIX: v <- (1 - lambda) v + lambda v_source of the same token, before it is cached */
+    /* retention in the pre-norm form: w_in rows q | k | v | g; act_qkv (UMBS_UNARY_* or 0) is applied to the q, k and v columns of the
+     * projection, keys are multiplied by k_scale (0 reads as dim^-1/2), rotary positions as in the parallel form; with out_norm_w
+     * (fp32 [heads vdim]) the concatenated heads are RMS-normed in norm_parts equal parts, times the weight, times the gate
+     * (gate_act: UMBS_GATE_*); without it: unit RMS per head times silu(g) */
+    int act_qkv;
+    float k_scale;
+    int gate_act;
+    /* latent attention in the pre-norm form with q_rank > 0: queries come through a normed latent of their own; w_in rows: dq (q_rank) |
+     * latent (kv_rank) | shared rotated key part (rope_dim) | gate (heads with gate_kind 1, heads vdim with gate_kind 2), w_uq
+     * [heads (dim + rope_dim), q_rank], q_norm [q_rank] */
 } umbs_layer_t;
 
 typedef struct {
@@ -263,6 +293,7 @@ typedef struct {
     const float* pos_freq;     /* fp32 [width / 2] or NULL: sinusoidal positions are added to the embedding,
                                 * entry 2i += sin(position pos_freq[i]), entry 2i + 1 += cos(position pos_freq[i]) */
     const float* embed_norm;   /* fp32 [width] or NULL: the embedding row is RMS-normed with this weight (goes with no pos_freq) */
+    float logit_scale;         /* factor on the logits, before the soft cap (0 reads as 1) */
 } umbs_model_t;
 
 const char* umbs_version(void);
@@ -316,6 +347,19 @@ int umbs_retention(int dtype, const float* qkvg, int64_t ld, const umbs_batch_t*
                    int rot_dims, const float* inv_freq, const float* decay, float eps, float* state, float* o_scratch,
                    float* rot_scratch, float* seg_scratch, size_t seg_bytes, void* out, umbs_stream_t stream);
 
+/* umbs_retention with the key factor and the output stage as arguments: keys times k_scale (0 reads as dim^-1/2); norm_w (fp32
+ * [heads vdim], or NULL: unit RMS per head times silu(g)): RMS norm in norm_parts equal parts of the concatenated heads times
+ * norm_w, times the gate (gate_act: UMBS_GATE_*). */
+typedef struct {
+    float k_scale;
+    const float* norm_w;
+    int norm_parts, gate_act;
+} umbs_retention_opts_t;
+int umbs_retention_ex(int dtype, const float* qkvg, int64_t ld, const umbs_batch_t* batch, int heads, int dim, int vdim,
+                      int rot_dims, const float* inv_freq, const float* decay, float eps, float* state, float* o_scratch,
+                      float* rot_scratch, float* seg_scratch, size_t seg_bytes, const umbs_retention_opts_t* opts, void* out,
+                      umbs_stream_t stream);
+
 /* Plain RMS norms of the two latents: x (fp32 [n, q_rank + kv_rank]) -> cq (`dtype` [n, q_rank]), c (`dtype` [n, kv_rank]). */
 int umbs_latent_norm(int dtype, const float* x, int n, int q_rank, int kv_rank, const float* q_norm, const float* kv_norm,
                      float eps, void* cq, void* c, umbs_stream_t stream);
@@ -358,6 +402,17 @@ int umbs_latent_prep(int dtype, const float* proj, int64_t ld, const umbs_batch_
                      int kv_rank, const float* kv_norm, float eps, int rot_dims, const float* inv_freq, float rot_mag, void* q,
                      void* c, float* q_rot, int64_t ld_qrot, umbs_stream_t stream);
 
+/* The pieces of umbs_latent_prep on their own, for queries that come through a latent: any of the three sources may be NULL.
+ * dq (fp32, row stride ld_dq) -> cq (`dtype` [n_tokens, q_rank]) = dq / rms(dq) * q_norm; low (fp32, row stride ld_low) =
+ * [latent | shared part] -> c; qsrc (fp32, row stride ld_q, heads (dim + rope_dim) numbers) -> q and q_rot, all as above. */
+typedef struct {
+    const float* dq; int64_t ld_dq; int q_rank; const float* q_norm; void* cq;
+    const float* low; int64_t ld_low; int kv_rank; const float* kv_norm; void* c;
+    const float* qsrc; int64_t ld_q; int heads, dim; void* q; float* q_rot; int64_t ld_qrot;
+    int rope_dim, rot_dims; const float* inv_freq; float rot_mag; float eps;
+} umbs_latent_prep_t;
+int umbs_latent_prep_parts(int dtype, const umbs_latent_prep_t* p, const umbs_batch_t* batch, umbs_stream_t stream);
+
 /* umbs_window_attention with options: k_shared (`dtype` [n_tokens, shared_dim], row stride ldks, or NULL) is a key part all
  * heads share -- a head's key is its own dim numbers of k followed by it, and q holds dim + shared_dim numbers per head;
  * window <= 0: every earlier token of the step; mode UMBS_ATTN_SOFTMAX_SINK: the denominator also holds exp(sink[head])
@@ -368,6 +423,12 @@ int umbs_window_attention_ex(int dtype, const void* q, int64_t ldq, const void* 
                              int64_t ldks, int shared_dim, const void* v, int64_t ldv, const umbs_batch_t* batch, int heads,
                              int dim, int vdim, int window, float scale, int mode, const float* sink, const float* gate,
                              int64_t ldg, void* out, int64_t ldo, umbs_stream_t stream);
+
+/* umbs_window_attention_ex with a gate per head: gate_per_head != 0 reads sigmoid(gate[t ldg + h]). */
+int umbs_window_attention_gated(int dtype, const void* q, int64_t ldq, const void* k, int64_t ldk, const void* k_shared,
+                                int64_t ldks, int shared_dim, const void* v, int64_t ldv, const umbs_batch_t* batch, int heads,
+                                int dim, int vdim, int window, float scale, int mode, const float* sink, const float* gate,
+                                int64_t ldg, int gate_per_head, void* out, int64_t ldo, umbs_stream_t stream);
 
 /* Stores this step's latents into the slots' rings (position p at row p mod ring_len). */
 int umbs_ring_append(int dtype, const void* c, void* ring, int ring_len, const umbs_batch_t* batch, int kv_rank,
@@ -503,6 +564,21 @@ int umbs_attention_prep_ex(int dtype, const float* proj, int64_t ld, const float
                            float* conv_state, int slots, int rot_dims, const float* inv_freq, float rot_mag, int maps,
                            const float* q_norm_w, const float* k_norm_w, float eps, void* q, void* kv, umbs_stream_t stream);
 
+/* umbs_attention_prep_ex with norms over a token's whole query and key rows and with mixed values. */
+typedef struct {
+    const float* q_norm_all_w; /* fp32 [heads maps dim] or NULL: RMS norm over all query numbers of the token at once (after bias and
+                                * convolution, before the rotation) */
+    const float* k_norm_all_w; /* fp32 [kv_heads maps dim] or NULL */
+    int v_mix;                 /* UMBS_VMIX_* */
+    float v_lambda;
+    float* v_source;           /* fp32 [n_tokens, kv_heads vdim]: written by UMBS_VMIX_SOURCE, read by UMBS_VMIX_MIX */
+} umbs_prep_opts_t;
+int umbs_attention_prep_opts(int dtype, const float* proj, int64_t ld, const float* bias, const umbs_batch_t* batch, int heads,
+                             int kv_heads, int dim, int vdim, int values_are_keys, int taps, const float* conv_w,
+                             float* conv_state, int slots, int rot_dims, const float* inv_freq, float rot_mag, int maps,
+                             const float* q_norm_w, const float* k_norm_w, float eps, const umbs_prep_opts_t* opts, void* q,
+                             void* kv, umbs_stream_t stream);
+
 /* Options of umbs_cached_attention_ex.  With maps = M and value_heads = C the kernel runs heads M C independent softmax rows
  * per token, numbered (h M + m) C + c: queries (h M + m) dim of q [n_tokens, heads M dim], keys ((h / rep) M + m) dim of a
  * key/value row [kv_heads M dim | kv_heads vdim], values of head c (C = kv_heads: every query head against every value
@@ -515,6 +591,7 @@ typedef struct {
     int maps;                  /* 0 reads as 1 */
     int value_heads;           /* 0 reads as 1 */
     float* raw_out;            /* fp32 [n_tokens, heads M C, vdim] or NULL: the normalised outputs go here (no gate) instead of out */
+    const float* sink;         /* fp32 [heads] or NULL: UMBS_ATTN_SOFTMAX_SINK with a score per head (NULL: 0) */
 } umbs_attn_opts_t;
 
 /* umbs_cached_attention with the options above (opts NULL: none).  Pooled blocks go with none of the options. */
@@ -587,10 +664,36 @@ int umbs_memory_run(const float* qkv, int64_t ld_qkv, const float* gates, const 
 int umbs_gated_norm(int dtype, const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w, int w_len,
                     int gate_first, float eps, void* out, umbs_stream_t stream);
 
+/* umbs_gated_norm with the gate's function as an argument (UMBS_GATE_*). */
+int umbs_gated_norm_ex(int dtype, const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w, int w_len,
+                       int gate_first, int gate_act, float eps, void* out, umbs_stream_t stream);
+
 /* umbs_gemm_ex for a plain product followed by a unary activation (UMBS_UNARY_*, with its two numbers). */
 int umbs_gemm_unary(int dtype, const void* A, int64_t lda, int a_goff, const void* W, int64_t ldw, int64_t w_gstride, void* C,
                     int64_t ldc, int c_goff, int c_f32, int M, int N, int K, int groups, const float* bias, int unary,
                     float p0, float p1, umbs_stream_t stream);
+
+/* umbs_gemm_unary on the first unary_cols output columns only (0: all of them). */
+int umbs_gemm_unary_cols(int dtype, const void* A, int64_t lda, int a_goff, const void* W, int64_t ldw, int64_t w_gstride, void* C,
+                         int64_t ldc, int c_goff, int c_f32, int M, int N, int K, int groups, const float* bias, int unary,
+                         float p0, float p1, int unary_cols, umbs_stream_t stream);
+
+/* umbs_gemm_ex whose gate is a number per row and group: the result is multiplied by sigmoid(out_gate[row ld_gate + g]). */
+int umbs_gemm_head_gate(int dtype, const void* A, int64_t lda, int a_goff, const void* W, int64_t ldw, int64_t w_gstride, void* C,
+                        int64_t ldc, int c_goff, int c_f32, int M, int N, int K, int groups, const float* out_gate,
+                        int64_t ld_gate, umbs_stream_t stream);
+
+/* Routing by token id, for all such layers of a model in one launch: what umbs_moe_route leaves, with the experts from
+ * table[ids[t]] and the weight 1 / top. */
+typedef struct {
+    const int32_t* table;      /* [vocab, top] */
+    int experts, top;
+    float* sel_w;              /* fp32 [n, top] */
+    int32_t* grp_off;          /* [experts + 1] */
+    int32_t* pair_tok;         /* [n top] */
+    int32_t* pair_pos;         /* [n top] */
+} umbs_table_route_t;
+int umbs_table_route(const int32_t* ids, int n, const umbs_table_route_t* layers, int n_layers, umbs_stream_t stream);
 
 /* umbs_moe_route_ex with a factor on the chosen weights; mode may also be UMBS_ROUTE_SOFTMAX_ALL. */
 int umbs_moe_route_scaled(int dtype, const void* h, int n, int width, const float* w_router, int experts, int top, int mode,
@@ -601,6 +704,10 @@ int umbs_moe_route_scaled(int dtype, const void* h, int n, int width, const floa
  * sin(tok_pos[t] pos_freq[i]), entry 2i + 1 the cosine; angles and sums in fp32. */
 int umbs_embedding_pos(int dtype, const int32_t* ids, const int32_t* tok_pos, const void* table, float scale,
                        const float* pos_freq, float* y, int n, int width, umbs_stream_t stream);
+
+/* umbs_embedding_pos that also leaves the row as `dtype` in y2 (row stride width; NULL: not). */
+int umbs_embedding_rows(int dtype, const int32_t* ids, const int32_t* tok_pos, const void* table, float scale,
+                        const float* pos_freq, float* y, void* y2, int n, int width, umbs_stream_t stream);
 
 int umbs_embedding(int dtype, const int32_t* ids, const void* table, float* y, int n, int width, umbs_stream_t stream);
 /* y[t] = table[ids[t]] * scale (fp32). */

@@ -22,8 +22,10 @@ UMBS_MEMORY_ADD, UMBS_MEMORY_DELTA = 0, 1
 UMBS_FORM_PARALLEL, UMBS_FORM_PRENORM = 0, 1
 UMBS_ACT_CLAMPED_GLU, UMBS_ACT_GELU_TANH, UMBS_ACT_SILU = 1, 2, 3
 UMBS_NORM_RMS, UMBS_NORM_LAYER, UMBS_NORM_DYT = 0, 1, 2
-UMBS_UNARY_TANH, UMBS_UNARY_XIELU = 1, 2
-UMBS_ROUTE_SOFTMAX_TOP, UMBS_ROUTE_SIGMOID_GROUPS, UMBS_ROUTE_SOFTMAX_ALL = 0, 1, 2
+UMBS_UNARY_TANH, UMBS_UNARY_XIELU, UMBS_UNARY_RELU2, UMBS_UNARY_SILU, UMBS_UNARY_SCALE = 1, 2, 3, 4, 5
+UMBS_GATE_SILU, UMBS_GATE_SIGMOID = 0, 1
+UMBS_VMIX_NONE, UMBS_VMIX_SOURCE, UMBS_VMIX_MIX = 0, 1, 2
+UMBS_ROUTE_SOFTMAX_TOP, UMBS_ROUTE_SIGMOID_GROUPS, UMBS_ROUTE_SOFTMAX_ALL, UMBS_ROUTE_TABLE = 0, 1, 2, 3
 UMBS_ATTN_SOFTMAX, UMBS_ATTN_SOFTMAX_SINK, UMBS_ATTN_SIGMOID = 0, 1, 2
 
 
@@ -39,7 +41,8 @@ class Mlp(C.Structure):
                 ("w_gu", c_void_p), ("w_down", c_void_p), ("shared_ff", c_int), ("shared_limit", c_float),
                 ("ws_gu", c_void_p), ("ws_down", c_void_p), ("act", c_int), ("route_mode", c_int), ("groups", c_int),
                 ("keep", c_int), ("bias_gu", c_void_p), ("bias_down", c_void_p), ("w_shared_gate", c_void_p),
-                ("route_scale", c_float), ("plain", c_int), ("unary", c_int), ("unary_p0", c_float), ("unary_p1", c_float)]
+                ("route_scale", c_float), ("plain", c_int), ("unary", c_int), ("unary_p0", c_float), ("unary_p1", c_float),
+                ("route_table", c_void_p)]
 
 
 class Delta(C.Structure):
@@ -73,7 +76,9 @@ Layer._fields_ = [("mixer", c_int), ("heads", c_int), ("dim", c_int), ("vdim", c
                 ("w_decay2", c_void_p), ("decay_bias", c_void_p), ("bonus", c_void_p), ("tm_state", c_void_p),
                 ("second", C.POINTER(Layer)), ("mix_scale", c_float), ("second_scale", c_float),
                 ("post_norm_w", c_void_p), ("post_norm2_w", c_void_p), ("w_merge", c_void_p), ("conv_b", c_void_p),
-                ("decay_rate", c_void_p), ("dt_bias", c_void_p), ("skip_w", c_void_p), ("norm_parts", c_int), ("mem_state", c_void_p)]
+                ("decay_rate", c_void_p), ("dt_bias", c_void_p), ("skip_w", c_void_p), ("norm_parts", c_int), ("mem_state", c_void_p),
+                ("q_norm_all_w", c_void_p), ("k_norm_all_w", c_void_p), ("v_mix", c_int), ("v_lambda", c_float),
+                ("act_qkv", c_int), ("k_scale", c_float), ("gate_act", c_int)]
 
 
 class Model(C.Structure):
@@ -81,12 +86,34 @@ class Model(C.Structure):
                 ("slots", c_int), ("norm_eps", c_float), ("embed", c_void_p), ("final_norm", c_void_p), ("head", c_void_p),
                 ("layers", C.POINTER(Layer)), ("norm_offset", c_float), ("logit_softcap", c_float),
                 ("embed_scale", c_float), ("norm_kind", c_int), ("final_norm_b", c_void_p), ("final_norm_alpha", c_float),
-                ("pos_freq", c_void_p), ("embed_norm", c_void_p)]
+                ("pos_freq", c_void_p), ("embed_norm", c_void_p), ("logit_scale", c_float)]
 
 
 class AttnOpts(C.Structure):
     _fields_ = [("softcap", c_float), ("dist_r1", c_void_p), ("dist_r2", c_void_p), ("chunk", c_int), ("maps", c_int),
-                ("value_heads", c_int), ("raw_out", c_void_p)]
+                ("value_heads", c_int), ("raw_out", c_void_p), ("sink", c_void_p)]
+
+
+class PrepOpts(C.Structure):
+    _fields_ = [("q_norm_all_w", c_void_p), ("k_norm_all_w", c_void_p), ("v_mix", c_int), ("v_lambda", c_float),
+                ("v_source", c_void_p)]
+
+
+class LatentPrep(C.Structure):
+    _fields_ = [("dq", c_void_p), ("ld_dq", c_int64), ("q_rank", c_int), ("q_norm", c_void_p), ("cq", c_void_p),
+                ("low", c_void_p), ("ld_low", c_int64), ("kv_rank", c_int), ("kv_norm", c_void_p), ("c", c_void_p),
+                ("qsrc", c_void_p), ("ld_q", c_int64), ("heads", c_int), ("dim", c_int), ("q", c_void_p), ("q_rot", c_void_p),
+                ("ld_qrot", c_int64), ("rope_dim", c_int), ("rot_dims", c_int), ("inv_freq", c_void_p), ("rot_mag", c_float),
+                ("eps", c_float)]
+
+
+class RetentionOpts(C.Structure):
+    _fields_ = [("k_scale", c_float), ("norm_w", c_void_p), ("norm_parts", c_int), ("gate_act", c_int)]
+
+
+class TableRoute(C.Structure):
+    _fields_ = [("table", c_void_p), ("experts", c_int), ("top", c_int), ("sel_w", c_void_p), ("grp_off", c_void_p),
+                ("pair_tok", c_void_p), ("pair_pos", c_void_p)]
 
 
 class Memory(C.Structure):
@@ -174,6 +201,24 @@ SIGNATURES = {
     "umbs_memory_run": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, C.POINTER(Memory), _BP, c_void_p, c_void_p]),
     "umbs_gated_norm": (c_int, [c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p,
                                 c_void_p]),
+    "umbs_attention_prep_opts": (c_int, [c_int, c_void_p, c_int64, c_void_p, _BP, c_int, c_int, c_int, c_int, c_int, c_int,
+                                         c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_int, c_void_p, c_void_p, c_float,
+                                         C.POINTER(PrepOpts), c_void_p, c_void_p, c_void_p]),
+    "umbs_latent_prep_parts": (c_int, [c_int, C.POINTER(LatentPrep), _BP, c_void_p]),
+    "umbs_window_attention_gated": (c_int, [c_int, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_void_p,
+                                            c_int64, _BP, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
+                                            c_int64, c_int, c_void_p, c_int64, c_void_p]),
+    "umbs_retention_ex": (c_int, [c_int, c_void_p, c_int64, _BP, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
+                                  c_void_p, c_void_p, c_void_p, c_void_p, c_size_t, C.POINTER(RetentionOpts), c_void_p, c_void_p]),
+    "umbs_gated_norm_ex": (c_int, [c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float,
+                                   c_void_p, c_void_p]),
+    "umbs_gemm_unary_cols": (c_int, [c_int, c_void_p, c_int64, c_int, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int, c_int,
+                                     c_int, c_int, c_int, c_int, c_void_p, c_int, c_float, c_float, c_int, c_void_p]),
+    "umbs_gemm_head_gate": (c_int, [c_int, c_void_p, c_int64, c_int, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int, c_int,
+                                    c_int, c_int, c_int, c_int, c_void_p, c_int64, c_void_p]),
+    "umbs_table_route": (c_int, [c_void_p, c_int, C.POINTER(TableRoute), c_int, c_void_p]),
+    "umbs_embedding_rows": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                    c_void_p]),
     "umbs_embedding": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]),
     "umbs_embedding_scaled": (c_int, [c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p]),
 }

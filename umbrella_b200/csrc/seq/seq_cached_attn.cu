@@ -39,7 +39,9 @@ struct CachedAttnArgs {
     void* out;
     // score options
     float softcap; const float* r1; const float* r2; int chunk, maps, vheads; float* raw;
+    const float* sink;                                // [heads] or NULL: the sink's score per head (NULL: 0)
 };
+__device__ __forceinline__ float sink_score(const CachedAttnArgs& a, int h) { return a.sink != nullptr ? a.sink[h] : 0.f; }
 
 // What a virtual head reads: its query's offset in a q row, its keys' and values' offsets in a key/value row.
 struct VHead { int h, qoff, koff, voff, row_kv, qstride, nv; };
@@ -95,9 +97,10 @@ __global__ void __launch_bounds__(256) cached_attention_kernel(CachedAttnArgs a,
         Qs[d * kCaS + r] = (q0 + r < len) ? to_f32(q[(int64_t)(start + q0 + r) * vhd.qstride + vhd.qoff + d]) : 0.f;
     }
     float m[4], l[4], o[4][VC];
+    const float sk = MODE == UMBS_ATTN_SOFTMAX_SINK ? sink_score(a, h) : -INFINITY;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-        m[i] = MODE == UMBS_ATTN_SOFTMAX_SINK ? 0.f : -INFINITY;       // the sink: a key of score 0 ...
+        m[i] = sk;                                                     // the sink: a key of this score ...
         l[i] = MODE == UMBS_ATTN_SOFTMAX_SINK ? 1.f : 0.f;             // ... that counts in the sum and has no value
 #pragma unroll
         for (int c = 0; c < VC; ++c) o[i][c] = 0.f;
@@ -383,13 +386,14 @@ __global__ void __launch_bounds__(32 * kCdWarps) cached_attention_decode_kernel(
             for (int ww = 0; ww < kCdWarps; ++ww) O += sm_o[ww][c];
     } else {
         for (int ww = 0; ww < kCdWarps; ++ww) M = fmaxf(M, sm_ml[ww][0]);
-        if (n_split == 1 && MODE == UMBS_ATTN_SOFTMAX_SINK) M = fmaxf(M, 0.f);
+        const float sk = (n_split == 1 && MODE == UMBS_ATTN_SOFTMAX_SINK) ? sink_score(a, h) : -INFINITY;
+        M = fmaxf(M, sk);
         for (int ww = 0; ww < kCdWarps; ++ww) {
             const float mw = sm_ml[ww][0], f = mw > -INFINITY ? expf(mw - M) : 0.f;
             L = fmaf(sm_ml[ww][1], f, L);
             if (c < vdim) O = fmaf(sm_o[ww][c], f, O);
         }
-        if (n_split == 1 && MODE == UMBS_ATTN_SOFTMAX_SINK) L += expf(-M);
+        if (n_split == 1 && MODE == UMBS_ATTN_SOFTMAX_SINK) L += expf(sk - M);
     }
     if (n_split > 1) {
         float* pr = part + (((int64_t)t * vhd.nv + vh) * n_split + split) * (vdim + 2);
@@ -412,7 +416,8 @@ __global__ void cached_attention_merge_kernel(CachedAttnArgs a, int n_split, con
     const int nv = a.heads * a.maps * a.vheads;
     const int th = blockIdx.x, t = th / nv, h = th - t * nv, vdim = a.vdim, c = threadIdx.x;      // (without options h is the head)
     const float* pr = part + (int64_t)th * n_split * (vdim + 2);
-    float M = MODE == UMBS_ATTN_SOFTMAX_SINK ? 0.f : -INFINITY, L = 0.f, O = 0.f;
+    const float sk = MODE == UMBS_ATTN_SOFTMAX_SINK ? sink_score(a, h / (a.maps * a.vheads)) : -INFINITY;
+    float M = sk, L = 0.f, O = 0.f;
     if (MODE == UMBS_ATTN_SIGMOID) {
         if (c < vdim)
             for (int i = 0; i < n_split; ++i) O += pr[i * (vdim + 2) + c];
@@ -423,7 +428,7 @@ __global__ void cached_attention_merge_kernel(CachedAttnArgs a, int n_split, con
             L = fmaf(pr[i * (vdim + 2) + vdim + 1], f, L);
             if (c < vdim) O = fmaf(pr[i * (vdim + 2) + c], f, O);
         }
-        if (MODE == UMBS_ATTN_SOFTMAX_SINK) L += expf(-M);
+        if (MODE == UMBS_ATTN_SOFTMAX_SINK) L += expf(sk - M);
     }
     if (c < vdim) {
         const float inv = MODE == UMBS_ATTN_SIGMOID ? 1.f : 1.f / L;
@@ -544,10 +549,11 @@ extern "C" int umbs_cached_attention_ex(int dtype, int mode, const void* q, cons
     if (dim < 1 || vdim < 1 || dim > 256 || vdim > 256) return UMB_ERR_UNSUPPORTED;      // tiles and lanes are sized for heads up to 256
     cudaStream_t st = (cudaStream_t)stream;
     CachedAttnArgs a{q, kv, kv_cache, pool_cache, kv_len, pool_len, heads, kv_heads, dim, vdim, window, pool, scale,
-                     head_bias, gate, ldg, gate_per_head, out, 0.f, nullptr, nullptr, 0, 1, 1, nullptr};
+                     head_bias, gate, ldg, gate_per_head, out, 0.f, nullptr, nullptr, 0, 1, 1, nullptr, nullptr};
     if (opts != nullptr) {
         a.softcap = opts->softcap; a.r1 = opts->dist_r1; a.r2 = opts->dist_r2; a.chunk = opts->chunk;
         a.maps = opts->maps > 0 ? opts->maps : 1; a.vheads = opts->value_heads > 0 ? opts->value_heads : 1; a.raw = opts->raw_out;
+        a.sink = opts->sink;
         const bool any = a.softcap > 0.f || a.r1 != nullptr || a.chunk > 0 || a.maps > 1 || a.vheads > 1;
         if ((a.r1 != nullptr) != (a.r2 != nullptr) || a.chunk < 0) return UMB_ERR_ARG;
         if (any && (pool > 0 || mode == UMBS_ATTN_SIGMOID)) return UMB_ERR_UNSUPPORTED;

@@ -64,6 +64,9 @@ struct Scratch {
     float* mem_qkv;    // fp32 [T, max channels]  a rank-one memory's convolved queries, keys and values
     float* mem_kq;     // fp32 [T, max kv_heads]  k . q
     void* merge;       // act [T, 2 width]  residual stream | embedding output in front of a looped pass
+    float* q32;        // fp32 [T, max heads (dim + rope_dim)]  queries from a latent, before their turn
+    float* v_src;      // fp32 [T, max kv_heads vdim]  the values later layers mix into theirs
+    std::vector<umbs_table_route_t> routes;   // per layer: routing by token id (table NULL: the layer has none)
     std::vector<void*> kv_rows;   // per layer: the step's key | value rows (a buffer of its own for a layer others borrow from)
 };
 
@@ -87,6 +90,7 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
     int hmax = 1, rotd = 1, in_rows = 1, hv = 1, qr = 1, kvr = 1, hd = 1, hkv = 1, hkvw = 1, top = 1, experts = 1, ff = 1, sff = 1;
     int hall = 1, cav = 1, rawd = 1, n_mix = 0, rank = 1, tmhd = 1;
     int memc = 0, memg = 0;
+    int q32w = 0, vsrc = 0;
     bool parallel = false, two = false, merges = false;
     auto up = [](int& a, int b) { if (b > a) a = b; };
     for (int i = 0; i < m->n_layers; ++i)
@@ -104,6 +108,7 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
             const int M = l.maps > 1 ? l.maps : 1;
             up(in_rows, l.heads * M * l.dim + l.kv_heads * M * l.dim + (l.values_are_keys ? 0 : l.kv_heads * l.vdim) + gate_rows);
             up(hd, l.heads * M * l.dim); up(hkvw, l.kv_heads * (M * l.dim + l.vdim)); up(cav, l.vdim);
+            if (l.v_mix != UMBS_VMIX_NONE) up(vsrc, l.kv_heads * l.vdim);
             up(rawd, l.heads * M * (l.talk != nullptr ? l.kv_heads : 1) * l.vdim);
         } else if (is_memory(l)) {
             up(in_rows, mem_channels(l) + l.heads * l.vdim + (l.mixer == UMBS_MIX_SSD ? 1 : 2) * l.heads);
@@ -124,9 +129,10 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
             if (T >= 128 && ent * plane > segb) segb = ent * plane;
         }
         else {
-            // (direct queries: q rows | latent | shared key part | gate rows; keys and queries carry rope_dim more numbers)
-            const int gate_rows = l.gate_kind == 2 ? l.heads * l.vdim : 0;
-            up(in_rows, l.q_rank > 0 ? l.q_rank + l.kv_rank : l.heads * (l.dim + l.rope_dim) + l.kv_rank + l.rope_dim + gate_rows);
+            // (q rows, or the query latent | latent | shared key part | gate rows; keys and queries carry rope_dim more numbers)
+            const int gate_rows = l.gate_kind == 1 ? l.heads : (l.gate_kind == 2 ? l.heads * l.vdim : 0);
+            up(in_rows, (l.q_rank > 0 ? l.q_rank : l.heads * (l.dim + l.rope_dim)) + l.kv_rank + l.rope_dim + gate_rows);
+            if (l.q_rank > 0 && l.form == UMBS_FORM_PRENORM) up(q32w, l.heads * (l.dim + l.rope_dim));
             up(hmax, l.heads); up(qr, l.q_rank); up(kvr, l.kv_rank + l.rope_dim); up(hd, l.heads * (l.dim + l.rope_dim));
             up(hkv, l.heads * (l.kv_rank + l.rope_dim));
             if (l.w_ukv != nullptr) up(hkvw, l.heads * (l.dim + l.rope_dim + l.vdim));
@@ -177,6 +183,19 @@ static size_t carve(const umbs_model_t* m, int T, int n_want, char* base, Scratc
     z.mem_qkv = (float*)a.take(Tz * memc * 4);
     z.mem_kq = (float*)a.take(Tz * memg * 4);
     z.merge = a.take(merges ? Tz * 2 * W * es : 0);
+    z.q32 = (float*)a.take(Tz * q32w * 4);
+    z.v_src = (float*)a.take(Tz * vsrc * 4);
+    z.routes.assign(m->n_layers, umbs_table_route_t{});
+    for (int i = 0; i < m->n_layers; ++i) {
+        const umbs_layer_t& l = m->layers[i];
+        if (!l.has_mlp || l.mlp.experts <= 0 || l.mlp.route_mode != UMBS_ROUTE_TABLE) continue;
+        umbs_table_route_t& r = z.routes[i];
+        r.table = l.mlp.route_table; r.experts = l.mlp.experts; r.top = l.mlp.top;
+        r.sel_w = (float*)a.take(Tz * r.top * 4);
+        r.grp_off = (int32_t*)a.take((size_t)(r.experts + 1) * 4);
+        r.pair_tok = (int32_t*)a.take(Tz * r.top * 4);
+        r.pair_pos = (int32_t*)a.take(Tz * r.top * 4);
+    }
     z.kv_rows.assign(m->n_layers, z.kv);
     for (int i = 0; i < m->n_layers; ++i) {
         const umbs_layer_t& l = m->layers[i];
@@ -213,13 +232,17 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
     const size_t es = dt == UMBS_F32 ? 4 : 2;
     bool merges = false;
     for (int i = 0; i < m->n_layers; ++i) merges |= m->layers[i].w_merge != nullptr;
+    // layers without a norm in front read the stream itself: the embedding leaves its rows in the activation dtype too
+    const bool raw_first = m->n_layers > 0 && m->layers[0].form == UMBS_FORM_PRENORM && m->layers[0].norm_w == nullptr && !merges &&
+                           m->embed_norm == nullptr;
     if (m->embed_norm != nullptr) {
         // (looped passes read the embedding output again: it waits in the second half of the merge rows)
         if (m->pos_freq != nullptr) return UMB_ERR_UNSUPPORTED;
         UMBS_TRY(umbs_embedding_norm(dt, b->tok_ids, m->embed, embed_scale, m->embed_norm, m->norm_eps, s.stack,
                                      merges ? (char*)s.merge + (size_t)W * es : nullptr, 2 * (int64_t)W, T, W, stream));
     } else {
-        UMBS_TRY(umbs_embedding_pos(dt, b->tok_ids, b->tok_pos, m->embed, embed_scale, m->pos_freq, s.stack, T, W, stream));
+        UMBS_TRY(umbs_embedding_rows(dt, b->tok_ids, b->tok_pos, m->embed, embed_scale, m->pos_freq, s.stack, raw_first ? s.h : nullptr, T,
+                                     W, stream));
         if (merges) UMBS_TRY(umbs_add_rows(dt, s.stack, nullptr, T, W, 0.f, (char*)s.merge + (size_t)W * es, 2 * (int64_t)W, nullptr, stream));
     }
     const float* x = s.stack;                    // layer 0 reads X_0 itself
@@ -228,6 +251,14 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
         if (i > 0 && m->layers[i].form != m->layers[0].form) return UMB_ERR_UNSUPPORTED;    // one form per model
         prenorm = m->layers[i].form == UMBS_FORM_PRENORM;
     }
+    // experts chosen by token id: every such layer's pair lists in one launch, before the first layer
+    std::vector<umbs_table_route_t> by_id;
+    for (int i = 0; i < m->n_layers; ++i) {
+        if (!m->layers[i].has_mlp || m->layers[i].mlp.experts <= 0 || m->layers[i].mlp.route_mode != UMBS_ROUTE_TABLE) continue;
+        if (!prenorm) return UMB_ERR_UNSUPPORTED;
+        by_id.push_back(s.routes[i]);
+    }
+    if (!by_id.empty()) UMBS_TRY(umbs_table_route(b->tok_ids, T, by_id.data(), (int)by_id.size(), stream));
     // Pre-norm layers: one fp32 residual stream, updated in place.  Every block's output waits in `pending` and is added
     // by the kernel that computes the next norm (or, behind the last layer, by the final norm).
     umbs_delta_t pend{};
@@ -235,6 +266,8 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
     // the residual add + norm in front of a block: the plain RMS kernel where nothing else is asked for
     auto norm_step = [&](const int32_t* rows, int n, int kind, const float* w, const float* bias, float off, float alpha,
                          void* y, float* copy) -> int {
+        if (w == nullptr && y != nullptr)       // no norm in front of the block: its input is the stream itself
+            return umbs_add_rows(dt, s.stack, has_pend ? &pend : nullptr, n, W, m->norm_eps, y, W, copy, stream);
         const bool plain = kind == UMBS_NORM_RMS && (!has_pend || (pend.pair_out == nullptr && pend.shared == nullptr &&
                                                                    pend.scale == nullptr && pend.mult == 1.f &&
                                                                    pend.delta2 == nullptr && pend.norm_w == nullptr && (pend.delta_mult == 0.f || pend.delta_mult == 1.f)));
@@ -259,10 +292,13 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
             void* kv_rows = s.kv_rows[src];
             const float* gate = gate_rows ? s.proj + cq + ck + cv : nullptr;
             UMBS_TRY(umbs_gemm(dt, s.h, W, 0, l.w_in, W, 0, s.proj, rows, 0, 1, T, rows, W, 1, nullptr, nullptr, 0, 0.f, stream));
-            UMBS_TRY(umbs_attention_prep_ex(dt, s.proj, rows, l.bias_in, b, l.heads, borrowed ? 0 : l.kv_heads, l.dim, l.vdim,
-                                            l.values_are_keys, l.taps, l.conv_w, l.conv_state, m->slots, l.rot_dims, l.inv_freq,
-                                            l.rot_mag, M, l.q_norm_w, l.k_norm_w, m->norm_eps, s.q, borrowed ? nullptr : kv_rows,
-                                            stream));
+            umbs_prep_opts_t po{};
+            po.q_norm_all_w = l.q_norm_all_w; po.k_norm_all_w = l.k_norm_all_w;
+            po.v_mix = l.v_mix; po.v_lambda = l.v_lambda; po.v_source = s.v_src;
+            UMBS_TRY(umbs_attention_prep_opts(dt, s.proj, rows, l.bias_in, b, l.heads, borrowed ? 0 : l.kv_heads, l.dim, l.vdim,
+                                              l.values_are_keys, l.taps, l.conv_w, l.conv_state, m->slots, l.rot_dims, l.inv_freq,
+                                              l.rot_mag, M, l.q_norm_w, l.k_norm_w, m->norm_eps, &po, s.q, borrowed ? nullptr : kv_rows,
+                                              stream));
             if (l.pool > 0)
                 UMBS_TRY(umbs_kv_pool(dt, kv_rows, l.kv_cache, l.kv_len, l.pool_cache, l.pool_len, b, row_kv, l.pool, stream));
             const bool finish = l.talk != nullptr || M > 1 || l.head_unit_norm || (l.out_mult != 0.f && l.out_mult != 1.f);
@@ -271,6 +307,7 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
             opts.softcap = l.softcap; opts.dist_r1 = l.dist_r1; opts.dist_r2 = l.dist_r2; opts.chunk = l.chunk; opts.maps = M;
             opts.value_heads = l.talk != nullptr ? l.kv_heads : 1;
             opts.raw_out = finish ? s.raw : nullptr;
+            opts.sink = l.sink;
             UMBS_TRY(umbs_cached_attention_ex(dt, l.attn_mode, s.q, kv_rows, l.kv_cache, l.kv_len, l.pool_cache, l.pool_len, b,
                                               l.heads, l.kv_heads, l.dim, l.vdim, l.window, l.pool, l.scale, l.head_bias,
                                               finish ? nullptr : gate, rows, l.gate_kind == 1, &opts, s.ca_part, s.ca_part_bytes,
@@ -331,7 +368,8 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
             has_pend = false;
             prev_out = nullptr;
         }
-        UMBS_TRY(norm_step(nullptr, T, l.norm_kind, l.norm_w, l.norm_b, l.norm_offset, l.norm_alpha, s.h, prev_out));
+        if (!(i == 0 && raw_first))
+            UMBS_TRY(norm_step(nullptr, T, l.norm_kind, l.norm_w, l.norm_b, l.norm_offset, l.norm_alpha, s.h, prev_out));
         const bool generic = l.mixer == UMBS_MIX_CACHED_ATTENTION || l.mixer == UMBS_MIX_TIME_MIX || is_memory(l);
         if (generic) {
             UMBS_TRY(run_mixer(l, i, s.mix_out));
@@ -352,24 +390,46 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
             UMBS_TRY(umbs_gemm(dt, s.h, W, 0, l.w_in, W, 0, s.proj, rows, 0, 1, T, rows, W, 1, nullptr, nullptr, 0, 0.f, stream));
             UMBS_TRY(umbs_mlstm(dt, s.proj, rows, l.bias_in, b, l.heads, l.dim, l.vdim, l.gate_cap, m->norm_eps, l.out_norm_w,
                                 l.mlstm_state, s.gates, s.o32, s.seg_bytes ? s.seg : nullptr, s.seg_bytes, s.mixed, stream));
+        } else if (l.mixer == UMBS_MIX_RETENTION) {
+            const int rows = 2 * l.heads * l.dim + 2 * hv;
+            UMBS_TRY(umbs_gemm_unary_cols(dt, s.h, W, 0, l.w_in, W, 0, s.proj, rows, 0, 1, T, rows, W, 1, nullptr, l.act_qkv, 0.f, 0.f,
+                                          rows - hv, stream));
+            umbs_retention_opts_t ro{};
+            ro.k_scale = l.k_scale; ro.norm_w = l.out_norm_w; ro.norm_parts = l.norm_parts > 0 ? l.norm_parts : 1; ro.gate_act = l.gate_act;
+            UMBS_TRY(umbs_retention_ex(dt, s.proj, rows, b, l.heads, l.dim, l.vdim, l.rot_dims, l.inv_freq, l.decay, m->norm_eps, l.ret_state,
+                                       s.o32, s.rot, s.seg_bytes ? s.seg : nullptr, s.seg_bytes, &ro, s.mixed, stream));
         } else if (l.mixer == UMBS_MIX_LATENT_ATTENTION) {
-            // direct queries, keys through one normed latent per token plus a rotated part all heads share
-            if (l.q_rank != 0 || l.gate_kind == 1 || l.w_ukT == nullptr || l.w_uv == nullptr) return UMB_ERR_UNSUPPORTED;
+            // queries direct or through a normed latent, keys through one normed latent per token plus a rotated part all heads share
+            if (l.w_ukT == nullptr || l.w_uv == nullptr) return UMB_ERR_UNSUPPORTED;
             const int Rt = l.rope_dim, hd1 = l.dim + Rt, hdq = l.heads * hd1, R = l.kv_rank, KD = R + Rt;
-            const int gate_rows = l.gate_kind == 2 ? hv : 0, rows = hdq + KD + gate_rows;
-            const float* gate = gate_rows ? s.proj + hdq + KD : nullptr;
+            const int head_gate = l.gate_kind == 1, gate_rows = head_gate ? l.heads : (l.gate_kind == 2 ? hv : 0);
+            const int q_rows = l.q_rank > 0 ? l.q_rank : hdq, rows = q_rows + KD + gate_rows;
+            const float* gate = gate_rows ? s.proj + q_rows + KD : nullptr;
             UMBS_TRY(umbs_gemm(dt, s.h, W, 0, l.w_in, W, 0, s.proj, rows, 0, 1, T, rows, W, 1, nullptr, nullptr, 0, 0.f, stream));
-            UMBS_TRY(umbs_latent_prep(dt, s.proj, rows, b, l.heads, l.dim, Rt, R, l.kv_norm, m->norm_eps, l.rot_dims, l.inv_freq,
-                                      l.rot_mag, s.q, s.c, s.q_abs + R, KD, stream));
+            umbs_latent_prep_t lp{};
+            lp.rope_dim = Rt; lp.rot_dims = l.rot_dims; lp.inv_freq = l.inv_freq; lp.rot_mag = l.rot_mag; lp.eps = m->norm_eps;
+            lp.low = s.proj + q_rows; lp.ld_low = rows; lp.kv_rank = R; lp.kv_norm = l.kv_norm; lp.c = s.c;
+            lp.heads = l.heads; lp.dim = l.dim; lp.q = s.q; lp.q_rot = s.q_abs + R; lp.ld_qrot = KD;
+            if (l.q_rank > 0) {
+                lp.dq = s.proj; lp.ld_dq = rows; lp.q_rank = l.q_rank; lp.q_norm = l.q_norm; lp.cq = s.cq;
+                UMBS_TRY(umbs_latent_prep_parts(dt, &lp, b, stream));
+                UMBS_TRY(umbs_gemm(dt, s.cq, l.q_rank, 0, l.w_uq, l.q_rank, 0, s.q32, hdq, 0, 1, T, hdq, l.q_rank, 1, nullptr, nullptr, 0,
+                                   0.f, stream));
+                lp.dq = nullptr; lp.low = nullptr;
+                lp.qsrc = s.q32; lp.ld_q = hdq;
+            } else {
+                lp.qsrc = s.proj; lp.ld_q = rows;
+            }
+            UMBS_TRY(umbs_latent_prep_parts(dt, &lp, b, stream));
             if (b->max_seq_len > 1 && b->max_pos0 == 0 && l.w_ukv != nullptr && umbs_window_attention_ex_fits(l.dim, Rt, l.vdim)) {
                 // a step of fresh sequences: every visible key is in the step, so every head's own key part and its values
                 // are up-projected once per token and a (row, key) pair costs dim + rope_dim + vdim multiply-adds
                 const int hdk = l.heads * l.dim;
                 UMBS_TRY(umbs_gemm(dt, s.c, KD, 0, l.w_ukv, R, 0, s.kv, hdk + hv, 0, 0, T, hdk + hv, R, 1, nullptr, nullptr, 0, 0.f,
                                    stream));
-                UMBS_TRY(umbs_window_attention_ex(dt, s.q, hdq, s.kv, hdk + hv, (const char*)s.c + (size_t)R * es, KD, Rt,
-                                                  (const char*)s.kv + (size_t)hdk * es, hdk + hv, b, l.heads, l.dim, l.vdim,
-                                                  l.window, l.scale, l.attn_mode, l.sink, gate, rows, s.mixed, hv, stream));
+                UMBS_TRY(umbs_window_attention_gated(dt, s.q, hdq, s.kv, hdk + hv, (const char*)s.c + (size_t)R * es, KD, Rt,
+                                                     (const char*)s.kv + (size_t)hdk * es, hdk + hv, b, l.heads, l.dim, l.vdim, l.window,
+                                                     l.scale, l.attn_mode, l.sink, gate, rows, head_gate, s.mixed, hv, stream));
                 UMBS_TRY(umbs_ring_append(dt, s.c, l.ring, l.ring_len, b, KD, stream));
             } else {
                 // q_abs[t, h, :R] = W_uk[h]^T q[t, h, :dim]: scores against the cached latents need no per-key up-projection;
@@ -380,8 +440,12 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
                                                   l.attn_mode, l.sink, s.la_part, s.la_part_bytes, s.o_lat, stream));
                 UMBS_TRY(umbs_ring_append(dt, s.c, l.ring, l.ring_len, b, KD, stream));
                 // values per head from the weighted latents, times the sigmoid output gate
-                UMBS_TRY(umbs_gemm_ex(dt, s.o_lat, (int64_t)l.heads * R, R, l.w_uv, R, (int64_t)l.vdim * R, s.mixed, hv, l.vdim, 0,
-                                      T, l.vdim, R, l.heads, nullptr, nullptr, 0, 0.f, nullptr, gate, rows, l.vdim, stream));
+                if (head_gate)
+                    UMBS_TRY(umbs_gemm_head_gate(dt, s.o_lat, (int64_t)l.heads * R, R, l.w_uv, R, (int64_t)l.vdim * R, s.mixed, hv,
+                                                 l.vdim, 0, T, l.vdim, R, l.heads, gate, rows, stream));
+                else
+                    UMBS_TRY(umbs_gemm_ex(dt, s.o_lat, (int64_t)l.heads * R, R, l.w_uv, R, (int64_t)l.vdim * R, s.mixed, hv, l.vdim, 0,
+                                          T, l.vdim, R, l.heads, nullptr, nullptr, 0, 0.f, nullptr, gate, rows, l.vdim, stream));
             }
         } else {
             return UMB_ERR_UNSUPPORTED;
@@ -401,21 +465,27 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
         has_pend = true;
         if (l.has_mlp) {
             const umbs_mlp_t& f = l.mlp;
-            if ((f.experts <= 0 && f.shared_ff <= 0) || l.norm2_w == nullptr) return UMB_ERR_UNSUPPORTED;
+            if ((f.experts <= 0 && f.shared_ff <= 0) || (l.norm2_w == nullptr) != (l.norm_w == nullptr)) return UMB_ERR_UNSUPPORTED;
             const int act = f.act ? f.act : UMBS_ACT_CLAMPED_GLU;
             UMBS_TRY(norm_step(nullptr, T, l.norm_kind, l.norm2_w, l.norm2_b, l.norm_offset, l.norm2_alpha, s.h, nullptr));
             pend = umbs_delta_t{};
             pend.scale = l.out_scale2; pend.mult = mult; pend.norm_w = l.post_norm2_w;
             if (f.experts > 0) {
-                // (the shared expert's per-token gate rides along as one more row of the router)
-                UMBS_TRY(umbs_moe_route_scaled(dt, s.h, T, W, f.w_router, f.experts, f.top, f.route_mode, f.groups, f.keep,
-                                               f.route_scale, s.sel_w, s.grp_off, s.pair_tok, s.pair_pos, s.route_scratch,
-                                               f.shared_ff > 0 ? f.w_shared_gate : nullptr, s.sgate, stream));
+                umbs_table_route_t r = s.routes[i];
+                if (f.route_mode == UMBS_ROUTE_TABLE) {          // (the lists were made before the first layer)
+                    if (f.shared_ff > 0 && f.w_shared_gate != nullptr) UMBS_TRY(umbs_token_gate(dt, s.h, T, W, f.w_shared_gate, s.sgate, stream));
+                } else {
+                    r.sel_w = s.sel_w; r.grp_off = s.grp_off; r.pair_tok = s.pair_tok; r.pair_pos = s.pair_pos;
+                    // (the shared expert's per-token gate rides along as one more row of the router)
+                    UMBS_TRY(umbs_moe_route_scaled(dt, s.h, T, W, f.w_router, f.experts, f.top, f.route_mode, f.groups, f.keep,
+                                                   f.route_scale, r.sel_w, r.grp_off, r.pair_tok, r.pair_pos, s.route_scratch,
+                                                   f.shared_ff > 0 ? f.w_shared_gate : nullptr, s.sgate, stream));
+                }
                 UMBS_TRY(umbs_gemm(dt, s.h, W, 0, f.w_gu, W, (int64_t)2 * f.ff * W, s.y, f.ff, 0, 0, T, f.ff, W, f.experts,
-                                   s.grp_off, s.pair_tok, act, f.limit, stream));
+                                   r.grp_off, r.pair_tok, act, f.limit, stream));
                 UMBS_TRY(umbs_gemm(dt, s.y, f.ff, 0, f.w_down, f.ff, (int64_t)W * f.ff, s.pair_out, W, 0, 1, T, W, f.ff, f.experts,
-                                   s.grp_off, nullptr, 0, 0.f, stream));
-                pend.pair_out = s.pair_out; pend.sel_w = s.sel_w; pend.pair_pos = s.pair_pos; pend.top = f.top;
+                                   r.grp_off, nullptr, 0, 0.f, stream));
+                pend.pair_out = s.pair_out; pend.sel_w = r.sel_w; pend.pair_pos = r.pair_pos; pend.top = f.top;
             }
             if (f.shared_ff > 0) {
                 if (f.plain)           // no gate rows: the activation of the up product alone, in its epilogue
@@ -444,13 +514,14 @@ extern "C" int umbs_forward(const umbs_model_t* m, const umbs_batch_t* b, float*
         if (logits != nullptr && b->n_want > 0) {
             UMBS_TRY(norm_step(b->want_rows, b->n_want, m->norm_kind, m->final_norm, m->final_norm_b, m->norm_offset,
                                m->final_norm_alpha, s.final_h, nullptr));
-            UMBS_TRY(umbs_gemm(dt, s.final_h, W, 0, m->head, W, 0, logits, m->vocab, 0, 1, b->n_want, m->vocab, W, 1, nullptr,
-                               nullptr, 0, 0.f, stream));
+            const bool scaled = m->logit_scale != 0.f && m->logit_scale != 1.f;
+            UMBS_TRY(umbs_gemm_unary(dt, s.final_h, W, 0, m->head, W, 0, logits, m->vocab, 0, 1, b->n_want, m->vocab, W, 1, nullptr,
+                                     scaled ? UMBS_UNARY_SCALE : 0, m->logit_scale, 0.f, stream));
             if (m->logit_softcap > 0.f) UMBS_TRY(umbs_softcap(logits, (int64_t)b->n_want * m->vocab, m->logit_softcap, stream));
         }
         return 0;
     }
-    if (merges) return UMB_ERR_UNSUPPORTED;
+    if (merges || (m->logit_scale != 0.f && m->logit_scale != 1.f)) return UMB_ERR_UNSUPPORTED;
     for (int i = 0; i < m->n_layers; ++i) {
         const umbs_layer_t& l = m->layers[i];
         UMBS_TRY(umbs_group_norm_shift(dt, x, l.norm_w, l.shift_w, l.shift_state, m->slots, b, W, m->norm_groups,

@@ -42,7 +42,7 @@ __device__ float block_sum(float v, float* red) {   // red: >= 33 floats of shar
 // (pos_freq != NULL: sinusoidal positions on top -- sine at the even entries, cosine at the odd ones, one frequency per pair)
 template <typename T>
 __global__ void embedding_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ y,
-                                 int width, float scale, const int32_t* __restrict__ tok_pos, const float* __restrict__ pos_freq) {
+                                 T* __restrict__ y2, int width, float scale, const int32_t* __restrict__ tok_pos, const float* __restrict__ pos_freq) {
     const int t = blockIdx.x;
     const T* row = table + (int64_t)ids[t] * width;
     const float pos = pos_freq != nullptr ? (float)tok_pos[t] : 0.f;
@@ -53,6 +53,7 @@ __global__ void embedding_kernel(const int32_t* __restrict__ ids, const T* __res
             v += (e & 1) ? cosf(ang) : sinf(ang);
         }
         y[(int64_t)t * width + e] = v;
+        if (y2 != nullptr) y2[(int64_t)t * width + e] = from_f32<T>(v);
     }
 }
 
@@ -159,7 +160,7 @@ template <int DPT, int kRetTB>
 __global__ void retention_kernel(const float* __restrict__ qkvg, int64_t ld, Batch b, int heads, int dim, int vdim,
                                  int rot_dims, const float* __restrict__ rot_tab, const float* __restrict__ inv_freq,
                                  const float* __restrict__ decay, float* __restrict__ state, float* __restrict__ o_out,
-                                 int seg_len, int n_seg, int pass, float* __restrict__ seg_state) {
+                                 float kscale, int seg_len, int n_seg, int pass, float* __restrict__ seg_state) {
     extern __shared__ __align__(16) float sm[];
     const int DS = blockDim.y, dimP = DS * DPT, nthr = 32 * DS;
     float* qs = sm;                          // [TB][dimP]
@@ -182,7 +183,6 @@ __global__ void retention_kernel(const float* __restrict__ qkvg, int64_t ld, Bat
     const bool col = j < vdim;
     const int64_t plane = (int64_t)heads * dim * vdim;
     const float dec = decay[h];
-    const float kscale = 1.f / sqrtf((float)dim);
     const int half = rot_dims / 2;
     float* st = state + (((int64_t)slot * heads + h) * dim) * vdim;
     const float* st_in = st;
@@ -732,6 +732,53 @@ __global__ void moe_scatter_kernel(const int32_t* __restrict__ sel_e, int n_pair
     pair_pos[i] = p;
 }
 
+// Routing by token id: one block per layer counts its pairs per expert, adds the counts up and hands the pairs out.  Nothing
+// here depends on the activations, so one launch at the start of a step serves every such layer of the model.
+constexpr int kTrLayers = 32;
+struct TableRouteArgs { umbs_table_route_t l[kTrLayers]; };
+__global__ void __launch_bounds__(1024) table_route_kernel(const int32_t* __restrict__ ids, int n, TableRouteArgs args) {
+    extern __shared__ int32_t cnt[];                 // [experts] counts, then [experts] next free places
+    __shared__ int32_t wsum[32];
+    const umbs_table_route_t r = args.l[blockIdx.x];
+    const int E = r.experts, pairs = n * r.top, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    int32_t* next = cnt + E;
+    for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
+    __syncthreads();
+#pragma unroll 4
+    for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(cnt + r.table[(int64_t)ids[i / r.top] * r.top + i % r.top], 1);
+    __syncthreads();
+    int base = 0;                                    // exclusive sums over the experts, a block's width at a time
+    for (int e0 = 0; e0 < E; e0 += blockDim.x) {
+        const int e = e0 + threadIdx.x, c = e < E ? cnt[e] : 0;
+        int inc = c;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int up = __shfl_up_sync(0xffffffffu, inc, o);
+            if (lane >= o) inc += up;
+        }
+        if (lane == 31) wsum[warp] = inc;
+        __syncthreads();
+        int before = 0, total = 0;
+        for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
+            if (w < warp) before += wsum[w];
+            total += wsum[w];
+        }
+        const int off = base + before + inc - c;
+        if (e < E) { next[e] = off; r.grp_off[e] = off; }
+        base += total;
+        __syncthreads();
+    }
+    if (threadIdx.x == 0) r.grp_off[E] = base;
+    const float wgt = 1.f / (float)r.top;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+        const int t = i / r.top, p = atomicAdd(next + r.table[(int64_t)ids[t] * r.top + (i - t * r.top)], 1);
+        r.pair_tok[p] = t;
+        r.pair_pos[i] = p;
+        r.sel_w[i] = wgt;
+    }
+}
+
 // One warp per token: g[t] = sigmoid(w . h[t]).
 template <typename T>
 __global__ void token_gate_kernel(const T* __restrict__ h, int n, int width, const float* __restrict__ w, float* __restrict__ g) {
@@ -798,10 +845,15 @@ extern "C" int umbs_embedding_scaled(int dtype, const int32_t* ids, const void* 
 
 extern "C" int umbs_embedding_pos(int dtype, const int32_t* ids, const int32_t* tok_pos, const void* table, float scale,
                                   const float* pos_freq, float* y, int n, int width, umbs_stream_t stream) {
+    return umbs_embedding_rows(dtype, ids, tok_pos, table, scale, pos_freq, y, nullptr, n, width, stream);
+}
+
+extern "C" int umbs_embedding_rows(int dtype, const int32_t* ids, const int32_t* tok_pos, const void* table, float scale,
+                                   const float* pos_freq, float* y, void* y2, int n, int width, umbs_stream_t stream) {
     if (n <= 0) return 0;
     if (pos_freq != nullptr && tok_pos == nullptr) return UMB_ERR_ARG;
     cudaStream_t st = (cudaStream_t)stream;
-    UMBS_DISPATCH_T(dtype, embedding_kernel<T><<<n, threads_for(width), 0, st>>>(ids, (const T*)table, y, width, scale, tok_pos,
+    UMBS_DISPATCH_T(dtype, embedding_kernel<T><<<n, threads_for(width), 0, st>>>(ids, (const T*)table, y, (T*)y2, width, scale, tok_pos,
                                                                               pos_freq));
     count_launches(1);
     return (int)cudaGetLastError();
@@ -846,7 +898,7 @@ extern "C" int umbs_group_norm_rows(int dtype, const float* x, const int32_t* ro
 template <int DPT, int kRetTB>
 static int launch_retention(const float* qkvg, int64_t ld, const Batch& b, int heads, int dim, int vdim, int rot_dims,
                             const float* rot_tab, const float* inv_freq, const float* decay, float* state, float* o,
-                            int seg_len, int n_seg, int pass, float* seg_state, cudaStream_t st) {
+                            float kscale, int seg_len, int n_seg, int pass, float* seg_state, cudaStream_t st) {
     const int ds = (dim + DPT - 1) / DPT;
     const dim3 grid(b.n_seqs * n_seg, heads, (vdim + 31) / 32), block(32, ds);
     const size_t smem = ((size_t)2 * kRetTB * ds * DPT + (size_t)ds * kRetTB * 32 + kRetTB * 32) * sizeof(float);
@@ -857,7 +909,7 @@ static int launch_retention(const float* qkvg, int64_t ld, const Batch& b, int h
         set = smem;
     }
     retention_kernel<DPT, kRetTB><<<grid, block, smem, st>>>(qkvg, ld, b, heads, dim, vdim, rot_dims, rot_tab, inv_freq, decay,
-                                                             state, o, seg_len, n_seg, pass, seg_state);
+                                                             state, o, kscale, seg_len, n_seg, pass, seg_state);
     return 0;
 }
 
@@ -865,7 +917,16 @@ extern "C" int umbs_retention(int dtype, const float* qkvg, int64_t ld, const um
                               int vdim, int rot_dims, const float* inv_freq, const float* decay, float eps, float* state,
                               float* o_scratch, float* rot_scratch, float* seg_scratch, size_t seg_bytes, void* out,
                               umbs_stream_t stream) {
+    return umbs_retention_ex(dtype, qkvg, ld, batch, heads, dim, vdim, rot_dims, inv_freq, decay, eps, state, o_scratch, rot_scratch,
+                             seg_scratch, seg_bytes, nullptr, out, stream);
+}
+
+extern "C" int umbs_retention_ex(int dtype, const float* qkvg, int64_t ld, const umbs_batch_t* batch, int heads, int dim,
+                                 int vdim, int rot_dims, const float* inv_freq, const float* decay, float eps, float* state,
+                                 float* o_scratch, float* rot_scratch, float* seg_scratch, size_t seg_bytes,
+                                 const umbs_retention_opts_t* opts, void* out, umbs_stream_t stream) {
     if (batch->n_tokens <= 0) return 0;
+    const float kscale = (opts != nullptr && opts->k_scale != 0.f) ? opts->k_scale : 1.f / sqrtf((float)dim);
     if (rot_dims < 0 || rot_dims > dim || (rot_dims & 1)) return UMB_ERR_ARG;
     cudaStream_t st = (cudaStream_t)stream;
     unsigned launches = 2;
@@ -892,9 +953,9 @@ extern "C" int umbs_retention(int dtype, const float* qkvg, int64_t ld, const um
         }
     }
     auto run = [&](int pass) -> int {
-        if (dim <= 32) return launch_retention<8, 16>(qkvg, ld, *batch, heads, dim, vdim, rot_dims, rot_tab, inv_freq, decay, state, o_scratch, seg_len, n_seg, pass, seg_scratch, st);
-        if (dim <= 128) return launch_retention<16, 16>(qkvg, ld, *batch, heads, dim, vdim, rot_dims, rot_tab, inv_freq, decay, state, o_scratch, seg_len, n_seg, pass, seg_scratch, st);
-        if (dim <= 512) return launch_retention<32, 8>(qkvg, ld, *batch, heads, dim, vdim, rot_dims, rot_tab, inv_freq, decay, state, o_scratch, seg_len, n_seg, pass, seg_scratch, st);
+        if (dim <= 32) return launch_retention<8, 16>(qkvg, ld, *batch, heads, dim, vdim, rot_dims, rot_tab, inv_freq, decay, state, o_scratch, kscale, seg_len, n_seg, pass, seg_scratch, st);
+        if (dim <= 128) return launch_retention<16, 16>(qkvg, ld, *batch, heads, dim, vdim, rot_dims, rot_tab, inv_freq, decay, state, o_scratch, kscale, seg_len, n_seg, pass, seg_scratch, st);
+        if (dim <= 512) return launch_retention<32, 8>(qkvg, ld, *batch, heads, dim, vdim, rot_dims, rot_tab, inv_freq, decay, state, o_scratch, kscale, seg_len, n_seg, pass, seg_scratch, st);
         return UMB_ERR_UNSUPPORTED;
     };
     int rc;
@@ -910,6 +971,12 @@ extern "C" int umbs_retention(int dtype, const float* qkvg, int64_t ld, const um
         rc = run(0);
     }
     if (rc) return rc;
+    if (opts != nullptr && opts->norm_w != nullptr) {
+        count_launches(launches - 1);
+        const int hv = heads * vdim;
+        return umbs_gated_norm_ex(dtype, o_scratch, qkvg + 2 * (int64_t)heads * dim + hv, ld, batch->n_tokens, hv, opts->norm_parts,
+                                  opts->norm_w, hv, 0, opts->gate_act, eps, out, stream);
+    }
     const int warps = batch->n_tokens * heads;
     UMBS_DISPATCH_T(dtype, retention_gate_kernel<T><<<(warps + 3) / 4, 128, 0, st>>>(o_scratch, qkvg, ld, batch->n_tokens,
                                                                                    heads, dim, vdim, eps, (T*)out));
@@ -1062,6 +1129,30 @@ extern "C" int umbs_moe_route_scaled(int dtype, const void* h, int n, int width,
     const int pairs = n * top;
     moe_scatter_kernel<<<(pairs + 255) / 256, 256, 0, st>>>(sel_e, pairs, top, grp_off, cursor, pair_tok, pair_pos);
     count_launches(3);
+    return (int)cudaGetLastError();
+}
+
+extern "C" int umbs_table_route(const int32_t* ids, int n, const umbs_table_route_t* layers, int n_layers, umbs_stream_t stream) {
+    if (n <= 0 || n_layers <= 0) return 0;
+    if (ids == nullptr || layers == nullptr) return UMB_ERR_ARG;
+    int experts = 1, most = 1;
+    for (int i = 0; i < n_layers; ++i) {
+        const umbs_table_route_t& l = layers[i];
+        if (l.table == nullptr || l.top < 1 || l.experts < l.top || l.sel_w == nullptr || l.grp_off == nullptr || l.pair_tok == nullptr ||
+            l.pair_pos == nullptr || (int64_t)n * l.top > 0x7fffffff)
+            return UMB_ERR_ARG;
+        if (l.experts > 4096) return UMB_ERR_UNSUPPORTED;       // two counters per expert in shared memory
+        experts = std::max(experts, l.experts);
+        most = std::max(most, l.top);
+    }
+    const int threads = std::min(1024, std::max(64, (std::max(n * most, experts) + 31) / 32 * 32));
+    for (int i0 = 0; i0 < n_layers; i0 += kTrLayers) {
+        TableRouteArgs args{};
+        const int k = std::min(kTrLayers, n_layers - i0);
+        for (int i = 0; i < k; ++i) args.l[i] = layers[i0 + i];
+        table_route_kernel<<<k, threads, (size_t)2 * experts * sizeof(int32_t), (cudaStream_t)stream>>>(ids, n, args);
+        count_launches(1);
+    }
     return (int)cudaGetLastError();
 }
 

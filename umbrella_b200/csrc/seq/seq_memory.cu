@@ -421,10 +421,11 @@ static int launch_memory(const float* qkv, int64_t ld, const float* gates, const
 }
 
 // ------------------------------------------------------------------------------------------------ gated norm
+__device__ __forceinline__ float gate_mem(float z, int act) { return act == UMBS_GATE_SIGMOID ? 1.f / (1.f + expf(-z)) : silu_mem(z); }
 // A warp (or, for long parts, a block) per part of a row.
 template <typename T>
 __global__ void gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int64_t ldg, int n_parts, int width, int parts,
-                                  const float* __restrict__ w, int w_len, int gate_first, float eps, int whole_block, T* __restrict__ out) {
+                                  const float* __restrict__ w, int w_len, int gate_first, int gate_act, float eps, int whole_block, T* __restrict__ out) {
     __shared__ float red[32];
     const int nw = blockDim.x >> 5, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int p = whole_block ? blockIdx.x : blockIdx.x * nw + warp;
@@ -435,7 +436,7 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const float* __re
     const float* grow = gate + (int64_t)t * ldg + e0;
     float ss = 0.f;
     for (int e = me; e < size; e += step) {
-        const float y = gate_first ? orow[e] * silu_mem(grow[e]) : orow[e];
+        const float y = gate_first ? orow[e] * gate_mem(grow[e], gate_act) : orow[e];
         ss = fmaf(y, y, ss);
     }
     ss = warp_sum_mem(ss);
@@ -446,14 +447,14 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const float* __re
     }
     const float inv = 1.f / sqrtf(ss / (float)size + eps);
     for (int e = me; e < size; e += step)
-        out[(int64_t)t * width + e0 + e] = from_f32<T>(orow[e] * silu_mem(grow[e]) * inv * w[(e0 + e) % w_len]);
+        out[(int64_t)t * width + e0 + e] = from_f32<T>(orow[e] * gate_mem(grow[e], gate_act) * inv * w[(e0 + e) % w_len]);
 }
 
 // The same in 16-byte pieces, a part's values held in registers (KEEP4 pieces per lane of the warp, or per thread of the block, that a
 // part has).
 template <typename T, int KEEP4>
 __global__ void gated_norm_vec_kernel(const float* __restrict__ o, const float* __restrict__ gate, int64_t ldg, int n_parts, int width, int parts,
-                                      const float* __restrict__ w, int w_len, int gate_first, float eps, int whole_block, T* __restrict__ out) {
+                                      const float* __restrict__ w, int w_len, int gate_first, int gate_act, float eps, int whole_block, T* __restrict__ out) {
     __shared__ float red[32];
     const int nw = blockDim.x >> 5, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int p = whole_block ? blockIdx.x : blockIdx.x * nw + warp;
@@ -472,7 +473,7 @@ __global__ void gated_norm_vec_kernel(const float* __restrict__ o, const float* 
     }
 #pragma unroll
     for (int i = 0; i < KEEP4; ++i) {
-        g[i] = make_float4(silu_mem(g[i].x), silu_mem(g[i].y), silu_mem(g[i].z), silu_mem(g[i].w));
+        g[i] = make_float4(gate_mem(g[i].x, gate_act), gate_mem(g[i].y, gate_act), gate_mem(g[i].z, gate_act), gate_mem(g[i].w, gate_act));
         const float4 v = make_float4(y[i].x * g[i].x, y[i].y * g[i].y, y[i].z * g[i].z, y[i].w * g[i].w);
         const float4 q = gate_first ? v : y[i];
         ss = fmaf(q.x, q.x, fmaf(q.y, q.y, fmaf(q.z, q.z, fmaf(q.w, q.w, ss))));
@@ -503,19 +504,19 @@ __global__ void gated_norm_vec_kernel(const float* __restrict__ o, const float* 
 
 template <typename T>
 static void launch_gated_norm(const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w, int w_len,
-                              int gate_first, float eps, T* out, cudaStream_t st) {
+                              int gate_first, int gate_act, float eps, T* out, cudaStream_t st) {
     const int size = width / parts, n_parts = n * parts;
     const uintptr_t ptrs = (uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out;
     if (size % 4 == 0 && ldg % 4 == 0 && w_len % 4 == 0 && ptrs % 16 == 0 && size <= 16384) {
         const int block = size > 512, threads = block ? ((size / 4 + 3) / 4 + 31) / 32 * 32 : 128;
         const unsigned grid = block ? n_parts : (n_parts + 3) / 4;
-        if (size <= 128) gated_norm_vec_kernel<T, 1><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
-        else if (size <= 256) gated_norm_vec_kernel<T, 2><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
-        else gated_norm_vec_kernel<T, 4><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, eps, block, out);
+        if (size <= 128) gated_norm_vec_kernel<T, 1><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, gate_act, eps, block, out);
+        else if (size <= 256) gated_norm_vec_kernel<T, 2><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, gate_act, eps, block, out);
+        else gated_norm_vec_kernel<T, 4><<<grid, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len, gate_first, gate_act, eps, block, out);
     } else {
         const int block = size > 256, threads = block ? (size >= 2048 ? 512 : 256) : 128;
         gated_norm_kernel<T><<<block ? n_parts : (n_parts + 3) / 4, threads, 0, st>>>(o, gate, ldg, n_parts, width, parts, w, w_len,
-                                                                                     gate_first, eps, block, out);
+                                                                                     gate_first, gate_act, eps, block, out);
     }
 }
 
@@ -596,11 +597,17 @@ extern "C" int umbs_memory_run(const float* qkv, int64_t ld_qkv, const float* ga
 
 extern "C" int umbs_gated_norm(int dtype, const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w,
                                int w_len, int gate_first, float eps, void* out, umbs_stream_t stream) {
+    return umbs_gated_norm_ex(dtype, o, gate, ldg, n, width, parts, w, w_len, gate_first, UMBS_GATE_SILU, eps, out, stream);
+}
+
+extern "C" int umbs_gated_norm_ex(int dtype, const float* o, const float* gate, int64_t ldg, int n, int width, int parts, const float* w,
+                                  int w_len, int gate_first, int gate_act, float eps, void* out, umbs_stream_t stream) {
     if (n <= 0) return 0;
+    if (gate_act != UMBS_GATE_SILU && gate_act != UMBS_GATE_SIGMOID) return UMB_ERR_ARG;
     if (o == nullptr || gate == nullptr || w == nullptr || out == nullptr || parts < 1 || width % parts != 0 || w_len < 1) return UMB_ERR_ARG;
     cudaStream_t st = (cudaStream_t)stream;
-    if (dtype == UMBS_BF16) launch_gated_norm(o, gate, ldg, n, width, parts, w, w_len, gate_first, eps, (__nv_bfloat16*)out, st);
-    else if (dtype == UMBS_F32) launch_gated_norm(o, gate, ldg, n, width, parts, w, w_len, gate_first, eps, (float*)out, st);
+    if (dtype == UMBS_BF16) launch_gated_norm(o, gate, ldg, n, width, parts, w, w_len, gate_first, gate_act, eps, (__nv_bfloat16*)out, st);
+    else if (dtype == UMBS_F32) launch_gated_norm(o, gate, ldg, n, width, parts, w, w_len, gate_first, gate_act, eps, (float*)out, st);
     else return UMB_ERR_ARG;
     count_launches(1);
     return (int)cudaGetLastError();

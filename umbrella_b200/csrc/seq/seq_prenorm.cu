@@ -192,9 +192,9 @@ __global__ void add_norm_kernel(float* __restrict__ x, umbs_delta_t d, int has_d
     }
 }
 
-// The common case of add_norm_kernel in 16-byte pieces: one dense pending output, with or without a norm of its own, and an
-// RMS norm (or none) of the sum.  KEEP4 pieces per thread; the block's sums as fixed trees, one barrier each (every warp adds
-// up the warps' partial sums itself).
+// The common cases of add_norm_kernel in 16-byte pieces: one dense pending output or the routed experts' rows (TOP > 0: that
+// many per token), with or without a norm of its own, times a number, and an RMS norm (or none) of the sum.  KEEP4 pieces per
+// thread; the block's sums as fixed trees, one barrier each (every warp adds up the warps' partial sums itself).
 __device__ __forceinline__ float block_sum_one_barrier(float v, float* red) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
     v = warp_sum_pn(v);
@@ -208,25 +208,45 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
 }
 
-template <typename T, int KEEP4>
-__global__ void add_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ post_w,
+template <typename T, int KEEP4, bool ROUTED>
+__global__ void add_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ sel_w,
+                                    const int32_t* __restrict__ pair_pos, int top, const float* __restrict__ post_w, float mult,
                                     const int32_t* __restrict__ rows, const float* __restrict__ w, float w_offset, int width, float eps,
                                     T* __restrict__ y, int64_t ldy, float* __restrict__ copy) {
     __shared__ float red[2][32];
     const int r = blockIdx.x, n4 = width / 4;
     const int64_t src = rows ? rows[r] : r;
     float4* xr = reinterpret_cast<float4*>(x + src * width);
-    const float4* dr = reinterpret_cast<const float4*>(delta + src * width);
     float4 v[KEEP4], d[KEEP4];
     float sum = 0.f;
 #pragma unroll
     for (int i = 0; i < KEEP4; ++i) {
         const int e = threadIdx.x + i * blockDim.x;
         v[i] = d[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (e < n4) { d[i] = dr[e]; v[i] = xr[e]; }
-        sum = fmaf(d[i].x, d[i].x, fmaf(d[i].y, d[i].y, fmaf(d[i].z, d[i].z, fmaf(d[i].w, d[i].w, sum))));
+        if (e < n4) {
+            v[i] = xr[e];
+            if (!ROUTED) d[i] = reinterpret_cast<const float4*>(delta + src * width)[e];
+        }
+    }
+    if (ROUTED) {                       // delta: the experts' output rows; the token's rows one after the other, two in flight
+#pragma unroll 2
+        for (int k = 0; k < top; ++k) {
+            const float wk = sel_w[src * top + k];
+            const float4* pr = reinterpret_cast<const float4*>(delta + (int64_t)pair_pos[src * top + k] * width);
+#pragma unroll
+            for (int i = 0; i < KEEP4; ++i) {
+                const int e = threadIdx.x + i * blockDim.x;
+                if (e < n4) {
+                    const float4 p = pr[e];
+                    d[i] = make_float4(fmaf(wk, p.x, d[i].x), fmaf(wk, p.y, d[i].y), fmaf(wk, p.z, d[i].z), fmaf(wk, p.w, d[i].w));
+                }
+            }
+        }
     }
     if (post_w != nullptr) {
+#pragma unroll
+        for (int i = 0; i < KEEP4; ++i)
+            sum = fmaf(d[i].x, d[i].x, fmaf(d[i].y, d[i].y, fmaf(d[i].z, d[i].z, fmaf(d[i].w, d[i].w, sum))));
         const float inv = 1.f / sqrtf(block_sum_one_barrier(sum, red[0]) / (float)width + eps);
 #pragma unroll
         for (int i = 0; i < KEEP4; ++i) {
@@ -240,7 +260,7 @@ __global__ void add_norm_vec_kernel(float* __restrict__ x, const float* __restri
     sum = 0.f;
 #pragma unroll
     for (int i = 0; i < KEEP4; ++i) {
-        v[i] = make_float4(v[i].x + d[i].x, v[i].y + d[i].y, v[i].z + d[i].z, v[i].w + d[i].w);
+        v[i] = make_float4(fmaf(mult, d[i].x, v[i].x), fmaf(mult, d[i].y, v[i].y), fmaf(mult, d[i].z, v[i].z), fmaf(mult, d[i].w, v[i].w));
         sum = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, sum))));
     }
     const float inv = w != nullptr ? 1.f / sqrtf(block_sum_one_barrier(sum, red[1]) / (float)width + eps) : 1.f;
@@ -261,15 +281,18 @@ __global__ void add_norm_vec_kernel(float* __restrict__ x, const float* __restri
     }
 }
 
-template <typename T>
+template <typename T, bool ROUTED>
 static void launch_add_norm_vec(float* x, const umbs_delta_t& d, const int32_t* rows, int n, const float* w, float w_offset, int width,
                                 float eps, T* y, int64_t ldy, float* copy, cudaStream_t st) {
     // few rows: spread each over as many threads as there are pieces; many: four pieces per thread
     const int n4 = width / 4, keep = n <= 148 ? (n4 <= 1024 ? 1 : 2) : 4;
     const int threads = ((n4 + keep - 1) / keep + 31) / 32 * 32;
-    if (keep == 1) add_norm_vec_kernel<T, 1><<<n, threads, 0, st>>>(x, d.delta, d.norm_w, rows, w, w_offset, width, eps, y, ldy, copy);
-    else if (keep == 2) add_norm_vec_kernel<T, 2><<<n, threads, 0, st>>>(x, d.delta, d.norm_w, rows, w, w_offset, width, eps, y, ldy, copy);
-    else add_norm_vec_kernel<T, 4><<<n, threads, 0, st>>>(x, d.delta, d.norm_w, rows, w, w_offset, width, eps, y, ldy, copy);
+    const float* delta = ROUTED ? d.pair_out : d.delta;
+#define UMBS_ANV(K) add_norm_vec_kernel<T, K, ROUTED><<<n, threads, 0, st>>>(x, delta, d.sel_w, d.pair_pos, d.top, d.norm_w, d.mult, rows, w, w_offset, width, eps, y, ldy, copy)
+    if (keep == 1) UMBS_ANV(1);
+    else if (keep == 2) UMBS_ANV(2);
+    else UMBS_ANV(4);
+#undef UMBS_ANV
 }
 
 // One block per token: the embedding row through an RMS norm, in fp32 and (for a product that reads it) as T.
@@ -292,44 +315,55 @@ __global__ void embedding_norm_kernel(const int32_t* __restrict__ ids, const T* 
     }
 }
 
-// One block per token of a latent-attention layer with direct queries: RMS norm of the latent, the turn of the shared key
-// part and of every head's rope part by the token's position.
+// One block per token of a latent-attention layer: RMS norms of the query latent and of the key latent, the turn of the shared key
+// part and of every head's rope part by the token's position; each where its source is given.
 template <typename T>
-__global__ void latent_prep_kernel(const float* __restrict__ proj, int64_t ld, Batch b, int heads, int dim, int rope, int R,
-                                   const float* __restrict__ kv_norm, float eps, int rot_dims, const float* __restrict__ inv_freq,
-                                   float rot_mag, T* __restrict__ q, T* __restrict__ c, float* __restrict__ q_rot, int64_t ld_qrot) {
+__global__ void latent_prep_kernel(umbs_latent_prep_t p, Batch b) {
     extern __shared__ float cs[];                 // cos | sin [rot_dims]
     __shared__ float red[33];
-    const int t = blockIdx.x, pos = b.tok_pos[t], half = rot_dims / 2, hd = dim + rope;
-    const float* row = proj + (int64_t)t * ld;
-    const float* low = row + (int64_t)heads * hd;
+    const int t = blockIdx.x, pos = b.tok_pos[t], half = p.rot_dims / 2, hd = p.dim + p.rope_dim;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        const float ang = (float)pos * inv_freq[i];
-        cs[i] = cosf(ang) * rot_mag;
-        cs[half + i] = sinf(ang) * rot_mag;
+        const float ang = (float)pos * p.inv_freq[i];
+        cs[i] = cosf(ang) * p.rot_mag;
+        cs[half + i] = sinf(ang) * p.rot_mag;
     }
-    float ss = 0.f;
-    for (int e = threadIdx.x; e < R; e += blockDim.x) ss = fmaf(low[e], low[e], ss);
-    ss = block_sum_pn(ss, red);                    // (its barriers also publish cs)
-    const float inv = 1.f / sqrtf(ss / (float)R + eps);
-    // the turn of component j of a rope part that starts at p
-    auto turned = [&](const float* p, int j) -> float {
-        if (j < half) return p[j] * cs[j] - p[j + half] * cs[half + j];
-        if (j < rot_dims) return p[j] * cs[j - half] + p[j - half] * cs[j];     // cs[j] = sin of pair j - half
-        return p[j];
+    // the turn of component j of a rope part that starts at r
+    auto turned = [&](const float* r, int j) -> float {
+        if (j < half) return r[j] * cs[j] - r[j + half] * cs[half + j];
+        if (j < p.rot_dims) return r[j] * cs[j - half] + r[j - half] * cs[j];     // cs[j] = sin of pair j - half
+        return r[j];
     };
-    T* crow = c + (int64_t)t * (R + rope);
-    for (int e = threadIdx.x; e < R; e += blockDim.x) crow[e] = from_f32<T>(low[e] * inv * kv_norm[e]);
-    for (int j = threadIdx.x; j < rope; j += blockDim.x) crow[R + j] = from_f32<T>(turned(low + R, j));
-    T* qrow = q + (int64_t)t * heads * hd;
-    for (int i = threadIdx.x; i < heads * hd; i += blockDim.x) {
-        const int h = i / hd, e = i - h * hd;
-        float o = row[i];
-        if (e >= dim) {
-            o = turned(row + (int64_t)h * hd + dim, e - dim);
-            if (q_rot != nullptr) q_rot[((int64_t)t * heads + h) * ld_qrot + (e - dim)] = o;
+    __syncthreads();
+    if (p.dq != nullptr) {
+        const float* row = p.dq + (int64_t)t * p.ld_dq;
+        float ss = 0.f;
+        for (int e = threadIdx.x; e < p.q_rank; e += blockDim.x) ss = fmaf(row[e], row[e], ss);
+        const float inv = 1.f / sqrtf(block_sum_pn(ss, red) / (float)p.q_rank + p.eps);
+        T* out = (T*)p.cq + (int64_t)t * p.q_rank;
+        for (int e = threadIdx.x; e < p.q_rank; e += blockDim.x) out[e] = from_f32<T>(row[e] * inv * p.q_norm[e]);
+    }
+    if (p.low != nullptr) {
+        const float* low = p.low + (int64_t)t * p.ld_low;
+        const int R = p.kv_rank;
+        float ss = 0.f;
+        for (int e = threadIdx.x; e < R; e += blockDim.x) ss = fmaf(low[e], low[e], ss);
+        const float inv = 1.f / sqrtf(block_sum_pn(ss, red) / (float)R + p.eps);
+        T* crow = (T*)p.c + (int64_t)t * (R + p.rope_dim);
+        for (int e = threadIdx.x; e < R; e += blockDim.x) crow[e] = from_f32<T>(low[e] * inv * p.kv_norm[e]);
+        for (int j = threadIdx.x; j < p.rope_dim; j += blockDim.x) crow[R + j] = from_f32<T>(turned(low + R, j));
+    }
+    if (p.qsrc != nullptr) {
+        const float* row = p.qsrc + (int64_t)t * p.ld_q;
+        T* qrow = (T*)p.q + (int64_t)t * p.heads * hd;
+        for (int i = threadIdx.x; i < p.heads * hd; i += blockDim.x) {
+            const int h = i / hd, e = i - h * hd;
+            float o = row[i];
+            if (e >= p.dim) {
+                o = turned(row + (int64_t)h * hd + p.dim, e - p.dim);
+                if (p.q_rot != nullptr) p.q_rot[((int64_t)t * p.heads + h) * p.ld_qrot + (e - p.dim)] = o;
+            }
+            qrow[i] = from_f32<T>(o);
         }
-        qrow[i] = from_f32<T>(o);
     }
 }
 
@@ -346,7 +380,7 @@ __global__ void attention_prep_kernel(const float* __restrict__ proj, int64_t ld
                                       const float* __restrict__ conv_w, float* __restrict__ conv_state, int slots, int rot_dims,
                                       const float* __restrict__ inv_freq, float rot_mag, int maps,
                                       const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float eps,
-                                      T* __restrict__ q_out, T* __restrict__ kv_out) {
+                                      umbs_prep_opts_t po, T* __restrict__ q_out, T* __restrict__ kv_out) {
     extern __shared__ float sm[];                 // [heads dim + kv_heads dim] convolved q | k, then cos | sin [rot_dims]
     const int Cq = heads * maps * dim, Ck = kv_heads * maps * dim, C = Cq + Ck, Cv = kv_heads * vdim;
     float* y = sm;
@@ -403,6 +437,29 @@ __global__ void attention_prep_kernel(const float* __restrict__ proj, int64_t ld
         }
         __syncthreads();
     }
+    if (po.q_norm_all_w != nullptr || po.k_norm_all_w != nullptr) {
+        // RMS norm over all of the token's query numbers, and over all of its key numbers
+        __shared__ float red[2][33];
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+        float sq = 0.f, sk = 0.f;
+        for (int c = threadIdx.x; c < C; c += blockDim.x) {
+            const float u = y[c];
+            if (c < Cq) sq = fmaf(u, u, sq);
+            else sk = fmaf(u, u, sk);
+        }
+        sq = warp_sum_pn(sq);
+        sk = warp_sum_pn(sk);
+        if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+        __syncthreads();
+        sq = warp_sum_pn(lane < nw ? red[0][lane] : 0.f);
+        sk = warp_sum_pn(lane < nw ? red[1][lane] : 0.f);
+        const float iq = 1.f / sqrtf(sq / (float)Cq + eps), ik = Ck > 0 ? 1.f / sqrtf(sk / (float)Ck + eps) : 0.f;
+        for (int c = threadIdx.x; c < C; c += blockDim.x) {
+            if (c < Cq) { if (po.q_norm_all_w != nullptr) y[c] = y[c] * iq * po.q_norm_all_w[c]; }
+            else if (po.k_norm_all_w != nullptr) y[c] = y[c] * ik * po.k_norm_all_w[c - Cq];
+        }
+        __syncthreads();
+    }
     const int row_kv = Ck + Cv;
     T* qo = q_out + (int64_t)t * Cq;
     T* ko = kv_out + (int64_t)t * row_kv;
@@ -421,7 +478,12 @@ __global__ void attention_prep_kernel(const float* __restrict__ proj, int64_t ld
         }
     }
     if (!values_are_keys && kv_out != nullptr)
-        for (int c = threadIdx.x; c < Cv; c += blockDim.x) ko[Ck + c] = from_f32<T>(row[C + c] + (bias ? bias[C + c] : 0.f));
+        for (int c = threadIdx.x; c < Cv; c += blockDim.x) {
+            float v = row[C + c] + (bias ? bias[C + c] : 0.f);
+            if (po.v_mix == UMBS_VMIX_SOURCE) po.v_source[(int64_t)t * Cv + c] = v;
+            else if (po.v_mix == UMBS_VMIX_MIX) v = (1.f - po.v_lambda) * v + po.v_lambda * po.v_source[(int64_t)t * Cv + c];
+            ko[Ck + c] = from_f32<T>(v);
+        }
 }
 
 // One block per (block of tokens completed by the step, sequence, 256 columns): the fp32 mean, in position order, of the
@@ -491,9 +553,13 @@ static int add_norm_run(int dtype, float* x, const umbs_delta_t* d, const int32_
     if (d != nullptr) dd = *d;
     if (dd.delta_mult == 0.f && dd.delta2 == nullptr) dd.delta_mult = 1.f;
     const uintptr_t ptrs = (uintptr_t)x | (uintptr_t)dd.delta | (uintptr_t)dd.norm_w | (uintptr_t)w | (uintptr_t)copy | (uintptr_t)y;
-    if (d != nullptr && dd.delta != nullptr && dd.pair_out == nullptr && dd.shared == nullptr && dd.delta2 == nullptr && dd.scale == nullptr &&
-        dd.mult == 1.f && dd.delta_mult == 1.f && (kind == UMBS_NORM_RMS || kind == kNormNone) && width % 4 == 0 && ldy % 4 == 0 && ptrs % 16 == 0)
-        UMBS_DISPATCH_T(dtype, launch_add_norm_vec<T>(x, dd, rows, n, kind == kNormNone ? nullptr : w, w_offset, width, eps, (T*)y, ldy, copy, st));
+    const bool vec = d != nullptr && dd.shared == nullptr && dd.delta2 == nullptr && dd.scale == nullptr && dd.delta_mult == 1.f &&
+                     (kind == UMBS_NORM_RMS || kind == kNormNone) && width % 4 == 0 && ldy % 4 == 0 && ptrs % 16 == 0;
+    const float* vw = kind == kNormNone ? nullptr : w;
+    if (vec && dd.delta != nullptr && dd.pair_out == nullptr)
+        UMBS_DISPATCH_T(dtype, (launch_add_norm_vec<T, false>(x, dd, rows, n, vw, w_offset, width, eps, (T*)y, ldy, copy, st)));
+    else if (vec && dd.delta == nullptr && dd.pair_out != nullptr && (uintptr_t)dd.pair_out % 16 == 0)
+        UMBS_DISPATCH_T(dtype, (launch_add_norm_vec<T, true>(x, dd, rows, n, vw, w_offset, width, eps, (T*)y, ldy, copy, st)));
     else
         UMBS_DISPATCH_T(dtype, add_norm_kernel<T><<<n, threads, 0, st>>>(x, dd, d != nullptr, rows, kind, w, b, w_offset, alpha, width,
                                                                          eps, (T*)y, ldy, copy));
@@ -535,12 +601,24 @@ extern "C" int umbs_latent_prep(int dtype, const float* proj, int64_t ld, const 
     if (heads < 1 || dim < 0 || rope_dim < 0 || kv_rank < 1 || rot_dims < 0 || rot_dims > rope_dim || (rot_dims & 1)) return UMB_ERR_ARG;
     if (rot_dims > 0 && inv_freq == nullptr) return UMB_ERR_ARG;
     if (proj == nullptr || kv_norm == nullptr || q == nullptr || c == nullptr) return UMB_ERR_ARG;
+    umbs_latent_prep_t p{};
+    p.low = proj + (int64_t)heads * (dim + rope_dim); p.ld_low = ld; p.kv_rank = kv_rank; p.kv_norm = kv_norm; p.c = c;
+    p.qsrc = proj; p.ld_q = ld; p.heads = heads; p.dim = dim; p.q = q; p.q_rot = q_rot; p.ld_qrot = ld_qrot;
+    p.rope_dim = rope_dim; p.rot_dims = rot_dims; p.inv_freq = inv_freq; p.rot_mag = rot_mag; p.eps = eps;
+    return umbs_latent_prep_parts(dtype, &p, batch, stream);
+}
+
+extern "C" int umbs_latent_prep_parts(int dtype, const umbs_latent_prep_t* p, const umbs_batch_t* batch, umbs_stream_t stream) {
+    if (batch->n_tokens <= 0) return 0;
+    if (p->rope_dim < 0 || p->rot_dims < 0 || p->rot_dims > p->rope_dim || (p->rot_dims & 1) || (p->rot_dims > 0 && p->inv_freq == nullptr)) return UMB_ERR_ARG;
+    if (p->dq == nullptr && p->low == nullptr && p->qsrc == nullptr) return UMB_ERR_ARG;
+    if (p->dq != nullptr && (p->q_rank < 1 || p->q_norm == nullptr || p->cq == nullptr)) return UMB_ERR_ARG;
+    if (p->low != nullptr && (p->kv_rank < 1 || p->kv_norm == nullptr || p->c == nullptr)) return UMB_ERR_ARG;
+    if (p->qsrc != nullptr && (p->heads < 1 || p->dim < 0 || p->q == nullptr)) return UMB_ERR_ARG;
     cudaStream_t st = (cudaStream_t)stream;
-    const int work = heads * (dim + rope_dim);
+    const int work = p->qsrc != nullptr ? p->heads * (p->dim + p->rope_dim) : (p->dq != nullptr ? p->q_rank : 0) + p->kv_rank + p->rope_dim;
     const int threads = work >= 4096 ? 512 : (work >= 1024 ? 256 : 128);
-    UMBS_DISPATCH_T(dtype, latent_prep_kernel<T><<<batch->n_tokens, threads, (size_t)(rot_dims + 2) * sizeof(float), st>>>(
-                               proj, ld, *batch, heads, dim, rope_dim, kv_rank, kv_norm, eps, rot_dims, inv_freq, rot_mag, (T*)q,
-                               (T*)c, q_rot, ld_qrot));
+    UMBS_DISPATCH_T(dtype, latent_prep_kernel<T><<<batch->n_tokens, threads, (size_t)(p->rot_dims + 2) * sizeof(float), st>>>(*p, *batch));
     count_launches(1);
     return (int)cudaGetLastError();
 }
@@ -567,6 +645,19 @@ extern "C" int umbs_attention_prep_ex(int dtype, const float* proj, int64_t ld, 
                                       const float* conv_w, float* conv_state, int slots, int rot_dims, const float* inv_freq,
                                       float rot_mag, int maps, const float* q_norm_w, const float* k_norm_w, float eps, void* q,
                                       void* kv, umbs_stream_t stream) {
+    return umbs_attention_prep_opts(dtype, proj, ld, bias, batch, heads, kv_heads, dim, vdim, values_are_keys, taps, conv_w, conv_state,
+                                    slots, rot_dims, inv_freq, rot_mag, maps, q_norm_w, k_norm_w, eps, nullptr, q, kv, stream);
+}
+
+extern "C" int umbs_attention_prep_opts(int dtype, const float* proj, int64_t ld, const float* bias, const umbs_batch_t* batch, int heads,
+                                        int kv_heads, int dim, int vdim, int values_are_keys, int taps, const float* conv_w,
+                                        float* conv_state, int slots, int rot_dims, const float* inv_freq, float rot_mag, int maps,
+                                        const float* q_norm_w, const float* k_norm_w, float eps, const umbs_prep_opts_t* opts, void* q,
+                                        void* kv, umbs_stream_t stream) {
+    umbs_prep_opts_t po{};
+    if (opts != nullptr) po = *opts;
+    if (po.v_mix < UMBS_VMIX_NONE || po.v_mix > UMBS_VMIX_MIX) return UMB_ERR_ARG;
+    if (po.v_mix != UMBS_VMIX_NONE && (po.v_source == nullptr || values_are_keys || kv_heads < 1)) return UMB_ERR_ARG;
     if (batch->n_tokens <= 0) return 0;
     if (maps < 1) maps = 1;
     if (rot_dims < 0 || rot_dims > dim || (rot_dims & 1) || taps < 1 || kv_heads < 0 || heads < 1) return UMB_ERR_ARG;
@@ -581,7 +672,7 @@ extern "C" int umbs_attention_prep_ex(int dtype, const float* proj, int64_t ld, 
     const int threads = batch->n_tokens <= 64 ? std::min(1024, (C + 31) / 32 * 32) : (C >= 1024 ? 256 : 128);
     UMBS_DISPATCH_T(dtype, attention_prep_kernel<T><<<batch->n_tokens, threads, smem, st>>>(
                                proj, ld, bias, *batch, heads, kv_heads, dim, vdim, values_are_keys, taps, conv_w, conv_state, slots,
-                               rot_dims, inv_freq, rot_mag, maps, q_norm_w, k_norm_w, eps, (T*)q, (T*)kv));
+                               rot_dims, inv_freq, rot_mag, maps, q_norm_w, k_norm_w, eps, po, (T*)q, (T*)kv));
     count_launches(1);
     return (int)cudaGetLastError();
 }

@@ -23,11 +23,11 @@ constexpr int kWaQ = 64, kWaK = 64, kWaS = 68;        // rows and keys per tile;
 // Options beside the plain form: a key part all heads share (ks: [n_tokens, sdim] with row stride ldks; a head's key is its
 // own dim numbers followed by the shared sdim, its query has dim + sdim numbers; here `dim` is that sum and `kdim` the head's
 // own part), a sink (a score without key or value that counts once in the sum: sink[h], or 0 without the array) and a
-// sigmoid gate per output element.
+// sigmoid gate per output element or per head.
 struct WindowExtra {
     const void* ks; int64_t ldks; int kdim;
     int use_sink; const float* sink;
-    const float* gate; int64_t ldg;
+    const float* gate; int64_t ldg; int gate_per_head;
 };
 
 template <typename T, int VC>
@@ -150,7 +150,8 @@ __global__ void __launch_bounds__(256) window_attention_kernel(const T* __restri
         if (r >= len) continue;
         const float inv = 1.f / l[i];
         T* orow = out + (int64_t)(start + r) * ldo + (int64_t)h * vdim;
-        const float* grow = x.gate ? x.gate + (int64_t)(start + r) * x.ldg + (int64_t)h * vdim : nullptr;
+        const float* grow = x.gate ? x.gate + (int64_t)(start + r) * x.ldg + (x.gate_per_head ? h : h * vdim) : nullptr;
+        const int gstep = x.gate_per_head ? 0 : 1;
 #pragma unroll
         for (int cb = 0; cb < VC / 4; ++cb)
 #pragma unroll
@@ -158,7 +159,7 @@ __global__ void __launch_bounds__(256) window_attention_kernel(const T* __restri
                 const int col = cb * 64 + tx * 4 + c;
                 if (col < vdim) {
                     float val = o[i][cb * 4 + c] * inv;
-                    if (grow != nullptr) val *= 1.f / (1.f + expf(-grow[col]));
+                    if (grow != nullptr) val *= 1.f / (1.f + expf(-grow[col * gstep]));
                     orow[col] = from_f32<T>(val);
                 }
             }
@@ -206,13 +207,22 @@ extern "C" int umbs_window_attention_ex(int dtype, const void* q, int64_t ldq, c
                                         int64_t ldks, int shared_dim, const void* v, int64_t ldv, const umbs_batch_t* batch,
                                         int heads, int dim, int vdim, int window, float scale, int mode, const float* sink,
                                         const float* gate, int64_t ldg, void* out, int64_t ldo, umbs_stream_t stream) {
+    return umbs_window_attention_gated(dtype, q, ldq, k, ldk, k_shared, ldks, shared_dim, v, ldv, batch, heads, dim, vdim, window, scale,
+                                       mode, sink, gate, ldg, 0, out, ldo, stream);
+}
+
+extern "C" int umbs_window_attention_gated(int dtype, const void* q, int64_t ldq, const void* k, int64_t ldk, const void* k_shared,
+                                           int64_t ldks, int shared_dim, const void* v, int64_t ldv, const umbs_batch_t* batch,
+                                           int heads, int dim, int vdim, int window, float scale, int mode, const float* sink,
+                                           const float* gate, int64_t ldg, int gate_per_head, void* out, int64_t ldo,
+                                           umbs_stream_t stream) {
     if (batch->n_tokens <= 0) return 0;
     if (heads < 1 || (shared_dim > 0 && k_shared == nullptr)) return UMB_ERR_ARG;
     if (mode != UMBS_ATTN_SOFTMAX && mode != UMBS_ATTN_SOFTMAX_SINK) return UMB_ERR_UNSUPPORTED;
     if (!umbs_window_attention_ex_fits(dim, shared_dim, vdim)) return UMB_ERR_UNSUPPORTED;
     if (window <= 0) window = 1 << 30;                       // every earlier token of the step
     cudaStream_t st = (cudaStream_t)stream;
-    const WindowExtra x{k_shared, ldks, dim, mode == UMBS_ATTN_SOFTMAX_SINK, sink, gate, ldg};
+    const WindowExtra x{k_shared, ldks, dim, mode == UMBS_ATTN_SOFTMAX_SINK, sink, gate, ldg, gate_per_head != 0};
     const int dq = dim + shared_dim;
     int rc;
     if (dtype == UMBS_BF16) {

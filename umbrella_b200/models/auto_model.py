@@ -69,9 +69,14 @@ def _ralapel(path, **kw):
     return ralapel.from_pretrained(path, **kw)
 
 
+def _revudra(path, **kw):
+    from . import revudra
+    return revudra.from_pretrained(path, **kw)
+
+
 # config.json ``architecture`` -> factory(path, device=, dtype=, max_length=, slots=, max_tokens=, ...)
 _ARCHITECTURES = {"Radanex": _radanex, "Zedotar": _zedotar, "Kulisun": _kulisun, "Subivik": _subivik,
-                  "Ralapel": _ralapel}
+                  "Ralapel": _ralapel, "Revudra": _revudra}
 
 
 def _make(model_name, offload=False, batch_size=1, max_length=None, device="cuda:0", dtype=torch.float16, **unused):

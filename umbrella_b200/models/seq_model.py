@@ -3,12 +3,13 @@
 A model is a ``SeqModelSpec``: width, vocabulary, the norm's constants and a list of ``SeqLayerSpec``s, each naming
 its form (``"parallel"``: one grouped norm feeds mixer and feed-forward side by side, with token shift and a depth
 average as options; ``"prenorm"``: x += mixer(norm1(x)), x += ff(norm2(x)), RMS or layer norms, optionally with a learned
-scale vector and a multiplier on every block's output), its mixer (``"retention"``, ``"latent_attention"``,
+scale vector, a norm of its own and a multiplier on every block's output, and optionally without the norms in front: the blocks
+then read x itself), its mixer (``"retention"``, ``"latent_attention"``,
 ``"cached_attention"``, ``"mlstm"``, ``"time_mix"``, ``"gated_delta"`` or ``"ssd"``) with that mixer's sizes and constants -- a pre-norm layer may run a
 second mixer beside the first (``second``), both reading the same normed rows --, and its feed-forward (routed experts and /
 or a shared expert -- a dense feed-forward is a shared expert alone -- or none).  A span of layers may run several times in a
 row with the same weights (``loop``), every run with state of its own.  Model families (models/radanex.py, models/zedotar.py,
-models/kulisun.py, models/subivik.py, models/ralapel.py) translate their config.json into a spec and their tensors into the per-layer
+models/kulisun.py, models/subivik.py, models/ralapel.py, models/revudra.py) translate their config.json into a spec and their tensors into the per-layer
 weight dicts ``load_layer`` takes; nothing below knows a family's names.
 
 One ``forward`` call runs a ragged batch: for every sequence its slot of the ``SequenceStateCache`` and its next
@@ -37,14 +38,16 @@ class SeqMlpSpec:
     shared_limit: float = 0.0
     act: str = "clamped_glu"          # or "gelu_tanh", "silu"
     route: str = "softmax_top"        # "softmax_top": the top logits, softmax over them | "sigmoid_groups": sigmoid
-                                      # scores, group-limited choice, chosen scores divided by their sum
+                                      # scores, group-limited choice, chosen scores divided by their sum | "table": the token id picks
+                                      # the experts, each with weight 1 / top (no router)
     groups: int = 1                   # sigmoid_groups: equal groups of neighbouring experts ...
     keep: int = 1                     # ... of which the best `keep` (by the sum of their two largest scores) stay eligible
     bias: bool = False                # the shared (dense) projections carry biases
     shared_gate: bool = False         # the shared expert's output is multiplied by sigmoid(w . h), a number per token
     route_scale: float = 1.0          # factor on the chosen experts' weights ("softmax_all": softmax over every expert, the
                                       # chosen scores as they are)
-    plain: str = ""                   # the dense part has no gate: W_down act(W_up h), act = "xielu" (two learned numbers)
+    plain: str = ""                   # the dense part has no gate: W_down act(W_up h), act = "xielu" (two learned numbers) or
+                                      # "relu2" (the square of relu)
 
 
 @dataclass
@@ -57,7 +60,12 @@ class SeqLayerSpec:
     rot_dims: int = 0
     rot_base: float = 10000.0
     decay: list = field(default_factory=list)
-    # latent attention (pre-norm form: q_rank 0 = queries straight from the layer input; also attn_mode, gate_kind 0 / 2,
+    qkv_act: str = ""                 # retention in the pre-norm form: activation of q, k and v ("silu" or none)
+    k_scale: float = 0.0              # ... factor on the keys (0: dim^-1/2)
+    out_norm: bool = False            # ... RMS norm with a weight over the concatenated heads (in norm_parts equal parts) and gate_act
+                                      # in place of the unit RMS per head and silu
+    gate_act: str = "silu"            # "silu" | "sigmoid"
+    # latent attention (pre-norm form: q_rank 0 = queries straight from the layer input; also attn_mode, gate_kind,
     # rot_dims <= rope_dim, inv_freq, rot_mag from below; window 0 = every earlier token)
     q_rank: int = 0
     kv_rank: int = 0
@@ -75,7 +83,7 @@ class SeqLayerSpec:
     bias: bool = False                # q, k, v projections carry biases
     head_bias: bool = False           # a number per head added to the scores
     rot_pairs: str = "halves"         # which dimensions turn together: "halves": i and i + rot_dims / 2 | "neighbours": 2i and
-                                      # 2i + 1 (latent attention with direct queries)
+                                      # 2i + 1 (latent attention in the pre-norm form)
     inv_freq: list | None = None      # rotary frequencies when they are not base^(-2i/rot_dims) (scaled forms)
     rot_mag: float = 1.0              # factor on cos and sin
     # cached attention, score options
@@ -87,6 +95,9 @@ class SeqLayerSpec:
     diff: float = 0.0                 # lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff; the output is scaled by 1 - diff
     head_unit_norm: bool = False      # every head's output is divided by its root mean square
     qk_norm: bool = False             # RMS norm (weight [dim]) of every query and key head (and map)
+    qk_norm_all: bool = False         # RMS norm over all of a token's query numbers at once (weight [heads dim]), and over its keys
+    v_mix: str = ""                   # "source": later layers mix this layer's values into theirs | "mix": v <- (1 - lambda) v +
+                                      # lambda v_source of the same token, lambda a learned number
     kv_from: int | None = None        # the layer has no key / value projections and reads that layer's keys and values
     # time mix (dim = vdim)
     decay_rank: int = 0
@@ -103,6 +114,7 @@ class SeqLayerSpec:
     form: str = "parallel"
     norm_offset: float = 0.0          # added to the layer's norm weights (1: weights stored around zero)
     norm_kind: str = "rms"            # pre-norm form: "rms" | "layer" (mean removed, weight and bias) | "dyt" (tanh(alpha x) w + b)
+    pre_norm: bool = True             # pre-norm form: False = no norms in front of the blocks, which read the stream itself
     post_norm: bool = False           # pre-norm form: an RMS norm behind every block, x += norm(block output)
     layer_scale: bool = False         # pre-norm form: every block's output is multiplied by a learned vector
     residual_mult: float = 1.0        # pre-norm form: x += residual_mult * block output
@@ -122,6 +134,7 @@ class SeqModelSpec:
     norm_offset: float = 0.0          # added to the final norm's weight
     logit_softcap: float = 0.0        # > 0: logits <- cap tanh(logits / cap)
     embed_scale: float = 1.0          # factor on the embedding rows
+    logit_scale: float = 1.0          # factor on the logits (before the soft cap)
     norm_kind: str = "rms"            # kind of the final norm (pre-norm form)
     pos_embed: str = ""               # "sinusoid": entry 2i of the embedding gets sin(p f_i), entry 2i + 1 cos(p f_i), ...
     pos_base: float = 10000.0         # ... f_i = pos_base^(-2i / width)
@@ -189,7 +202,11 @@ _ATTN_MODES = {"softmax": S.UMBS_ATTN_SOFTMAX, "softmax_sink": S.UMBS_ATTN_SOFTM
 _ACTS = {"clamped_glu": S.UMBS_ACT_CLAMPED_GLU, "gelu_tanh": S.UMBS_ACT_GELU_TANH, "silu": S.UMBS_ACT_SILU}
 _NORMS = {"rms": S.UMBS_NORM_RMS, "layer": S.UMBS_NORM_LAYER, "dyt": S.UMBS_NORM_DYT}
 _ROUTES = {"softmax_top": S.UMBS_ROUTE_SOFTMAX_TOP, "sigmoid_groups": S.UMBS_ROUTE_SIGMOID_GROUPS,
-           "softmax_all": S.UMBS_ROUTE_SOFTMAX_ALL}
+           "softmax_all": S.UMBS_ROUTE_SOFTMAX_ALL, "table": S.UMBS_ROUTE_TABLE}
+_QKV_ACTS = {"": 0, "silu": S.UMBS_UNARY_SILU}
+_GATE_ACTS = {"silu": S.UMBS_GATE_SILU, "sigmoid": S.UMBS_GATE_SIGMOID}
+_PLAIN_ACTS = {"xielu": S.UMBS_UNARY_XIELU, "relu2": S.UMBS_UNARY_RELU2}
+_V_MIXES = {"": S.UMBS_VMIX_NONE, "source": S.UMBS_VMIX_SOURCE, "mix": S.UMBS_VMIX_MIX}
 
 
 def pair_rows_as_halves(w: torch.Tensor, first: int, rot_dims: int) -> torch.Tensor:
@@ -227,6 +244,15 @@ class SeqStateModel:
                 raise ValueError("loop: 0 <= start < stop <= layers and at least one pass")
             if any(l.form != "prenorm" or l.kv_from is not None for l in spec.layers):
                 raise ValueError("a loop goes with pre-norm layers that keep their own keys and values")
+        source = None                       # the layer whose values later ones mix in
+        for l in spec.layers:
+            if l.v_mix not in _V_MIXES or (l.v_mix and (l.mixer != "cached_attention" or l.kv_from is not None or l.values_are_keys or
+                                                        l.second is not None or spec.loop is not None)):
+                raise ValueError("mixed values go with cached attention over values of its own, one run and one mixer per layer")
+            if l.v_mix == "source":
+                source = l
+            elif l.v_mix == "mix" and (source is None or source.kv_heads * source.vdim != l.kv_heads * l.vdim):
+                raise ValueError("a layer that mixes values needs an earlier source layer with as many value numbers")
         self.eos_tokens = list(spec.eos_token_id)
         self._slots0, self._max_tokens0 = slots, max_tokens
         self.weights: list[dict | None] = [None] * self.num_layers
@@ -295,28 +321,33 @@ class SeqStateModel:
 
     def load_layer(self, idx: int, w: dict):
         """``w``: tensors [out, in] as the checkpoint holds them.
-        all layers: norm [width]; shift [width] (if the layer shifts); depth [idx + 2] (if it averages); o.
+        all layers: norm [width] (unless pre_norm is off); shift [width] (if the layer shifts); depth [idx + 2] (if it averages); o.
         retention: q, k [heads dim, width]; v, g [heads vdim, width].
         latent attention: dq [q_rank, width], dq_norm, uq [heads dim, q_rank], dkv [kv_rank, width], dkv_norm,
             uk [heads dim, kv_rank], uv [heads vdim, kv_rank].
+        retention in the pre-norm form: also out_norm [heads vdim] (with out_norm).
         cached attention: q [heads dim, width], k [kv_heads dim, width], v [kv_heads vdim, width] (unless the values are
             the keys), g [heads or heads vdim, width] (by gate_kind); q_b, k_b, v_b (biases); q_conv, k_conv [channels, taps];
-            pb [heads] (score bias).
+            pb [heads] (score bias); sink [heads] (learned_sink); q_norm, k_norm [heads dim], [kv_heads dim] (qk_norm_all); vmix (one
+            number, v_mix "mix").
         mlstm: q, k [heads dim, width]; v, g [heads vdim, width]; i, f [heads, width] with i_b, f_b [heads]; out_norm [heads vdim].
         latent attention with direct queries (q_rank 0): q [heads (dim + rope_dim), width], dkv [kv_rank + rope_dim, width],
-            dkv_norm, uk, uv, g [heads vdim, width] (gate_kind 2), sink [heads] (learned_sink).
+            dkv_norm, uk, uv, g [heads vdim, width] (gate_kind 2; [heads, width]: 1), sink [heads] (learned_sink); in the pre-norm form
+            with q_rank > 0: dq [q_rank, width], dq_norm, uq [heads (dim + rope_dim), q_rank] in place of q.
         gated delta: q, k [kv_heads dim, width]; v, g [heads vdim, width]; b, a [heads, width]; q_conv, k_conv, v_conv [channels, taps];
             A_log, dt_bias [heads]; out_norm [vdim].
         state space: in [2 heads vdim + 2 kv_heads dim + heads, width] (gate | v | k | q | step size); conv [channels of v | k | q, taps],
             conv_b; A_log, dt_bias, D [heads]; out_norm [heads vdim].
         pre-norm layers: post_norm, post_norm2 [width] (norms behind the blocks); norm2 [width] when they have a feed-forward; norm_b, norm2_b (layer norm); ls1, ls2 [width] (layer scale).
-        feed-forward: router [experts, width]; experts: list of (gate, up, down); shared (or dense): (gate, up, down);
+        feed-forward: router [experts, width] or (route "table") table [vocab, top] integers; experts: list of (gate, up, down); shared (or dense): (gate, up, down);
             dense_b: (gate_b, up_b, down_b) with ``bias``; shared_gate [1, width] or [width]."""
         l = self.spec.layers[idx]
-        d = dict(norm=self._f32(w["norm"]))
+        d = dict(norm=self._f32(w["norm"])) if l.pre_norm else {}
+        if not l.pre_norm and (l.form != "prenorm" or l.norm_kind != "rms"):
+            raise ValueError("layers without norms in front are of the pre-norm form, with RMS norms")
         if l.form == "prenorm":
             l.shift = l.depth_average = False
-            if l.mlp is not None:
+            if l.mlp is not None and l.pre_norm:
                 d["norm2"] = self._f32(w["norm2"])
             if l.norm_kind in ("layer", "dyt"):
                 d["norm_b"] = self._f32(w["norm_b"])
@@ -358,17 +389,26 @@ class SeqStateModel:
                 torch.zeros(1, dtype=torch.float32, device=self.device)
             d["decay"] = torch.tensor([float(x) for x in l.decay], dtype=torch.float32, device=self.device)
             assert d["decay"].numel() == l.heads and d["w_in"].shape == (2 * l.heads * (l.dim + l.vdim), self.spec.width)
-        elif l.mixer == "latent_attention" and l.q_rank == 0:
+            if l.form != "prenorm" and (l.qkv_act or l.k_scale or l.out_norm):
+                raise ValueError("retention's activation, key factor and norm over the heads are options of the pre-norm form")
+            if l.out_norm:
+                d["out_norm"] = self._f32(w["out_norm"])
+                assert d["out_norm"].numel() == l.heads * l.vdim and l.heads * l.vdim % l.norm_parts == 0
+        elif l.mixer == "latent_attention" and (l.q_rank == 0 or l.form == "prenorm"):
             if l.form != "prenorm":
                 raise ValueError("latent attention with direct queries is a pre-norm mixer")
             hd1 = l.dim + l.rope_dim
-            wq, wdkv = w["q"], w["dkv"]
+            wq, wdkv = w["uq" if l.q_rank else "q"], w["dkv"]
+            assert wq.shape == (l.heads * hd1, l.q_rank or self.spec.width) and wdkv.shape == (l.kv_rank + l.rope_dim, self.spec.width)
             if l.rot_pairs == "neighbours" and l.rot_dims:
                 wq = pair_rows_as_halves(wq.reshape(l.heads, hd1, -1), l.dim, l.rot_dims).reshape(wq.shape)
                 wdkv = pair_rows_as_halves(wdkv, l.kv_rank, l.rot_dims)
             elif l.rot_pairs not in ("halves", "neighbours"):
                 raise ValueError(f"unknown rotary pairing '{l.rot_pairs}'")
-            d["w_in"] = self._act(torch.cat([wq, wdkv] + ([w["g"]] if l.gate_kind else []), dim=0))
+            d["w_in"] = self._act(torch.cat([w["dq"] if l.q_rank else wq, wdkv] + ([w["g"]] if l.gate_kind else []), dim=0))
+            if l.q_rank:
+                d["q_norm"], d["uq"] = self._f32(w["dq_norm"]), self._act(wq)
+                assert w["dq"].shape == (l.q_rank, self.spec.width) and d["q_norm"].numel() == l.q_rank
             d["kv_norm"] = self._f32(w["dkv_norm"])
             d["ukT"] = self._act(w["uk"].reshape(l.heads, l.dim, l.kv_rank).transpose(1, 2))
             d["uv"] = self._act(w["uv"])
@@ -380,9 +420,9 @@ class SeqStateModel:
                 rotary_inv_freq64(l.rot_dims, l.rot_base) if l.rot_dims else None
             d["inv_freq"] = f.to(torch.float32).to(self.device) if l.rot_dims else \
                 torch.zeros(1, dtype=torch.float32, device=self.device)
-            assert w["q"].shape == (l.heads * hd1, self.spec.width) and w["dkv"].shape == (l.kv_rank + l.rope_dim, self.spec.width)
             assert w["uk"].shape == (l.heads * l.dim, l.kv_rank) and d["uv"].shape == (l.heads * l.vdim, l.kv_rank)
-            assert l.gate_kind in (0, 2) and (not l.gate_kind or w["g"].shape[0] == l.heads * l.vdim)
+            assert not l.gate_kind or w["g"].shape[0] == (l.heads if l.gate_kind == 1 else l.heads * l.vdim)
+            assert not l.learned_sink or d["sink"].numel() == l.heads
             assert l.rot_dims % 2 == 0 and l.rot_dims <= l.rope_dim and (not l.rot_dims or d["inv_freq"].numel() == l.rot_dims // 2)
         elif l.mixer == "latent_attention":
             d["w_in"] = self._act(torch.cat([w["dq"], w["dkv"]], dim=0))
@@ -415,6 +455,17 @@ class SeqStateModel:
                 if own:
                     d["k_norm"] = self._f32(w["k_norm"])
                 assert d["q_norm"].numel() == l.dim
+            if l.qk_norm_all:
+                d["q_norm_all"] = self._f32(w["q_norm"])
+                assert not l.qk_norm and d["q_norm_all"].numel() == cq
+                if own:
+                    d["k_norm_all"] = self._f32(w["k_norm"])
+                    assert d["k_norm_all"].numel() == ck
+            if l.learned_sink:
+                d["sink"] = self._f32(w["sink"])
+                assert d["sink"].numel() == l.heads and l.attn_mode == "softmax_sink"
+            if l.v_mix == "mix":
+                d["v_lambda"] = float(w["vmix"].double().reshape(()))
             if l.maps == 2:        # one number per layer, from four learned vectors: evaluated once, in double
                 dot = lambda a, b: float((w[a].double() * w[b].double()).sum())
                 d["diff_lambda"] = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + l.diff
@@ -474,16 +525,25 @@ class SeqStateModel:
         if l.mlp is not None:
             m = l.mlp
             if m.plain:
-                if m.plain != "xielu" or m.experts or l.form != "prenorm":
-                    raise ValueError("a plain feed-forward is W_down xielu(W_up h) of a pre-norm layer")
+                if m.plain not in _PLAIN_ACTS or m.experts or l.form != "prenorm":
+                    raise ValueError("a plain feed-forward is W_down act(W_up h) of a pre-norm layer, act = xielu or relu2")
                 up, dn = w["dense"]
                 d["s_gu"], d["s_down"] = self._act(up), self._act(dn)
-                p, q = (float(x) for x in w["dense_act"].double().reshape(-1))
-                d["unary_p"] = (_softplus(p), 0.5 + _softplus(q))        # the two coefficients, evaluated once in double
+                if m.plain == "xielu":
+                    p, q = (float(x) for x in w["dense_act"].double().reshape(-1))
+                    d["unary_p"] = (_softplus(p), 0.5 + _softplus(q))        # the two coefficients, evaluated once in double
                 assert d["s_gu"].shape == (m.shared_ff, self.spec.width) and d["s_down"].shape == (self.spec.width, m.shared_ff)
                 return
             if m.experts:
-                d["router"] = self._f32(w["router"])
+                if m.route == "table":
+                    if l.form != "prenorm":
+                        raise ValueError("experts chosen by token id go with pre-norm layers")
+                    t = w["table"]
+                    if t.shape != (self.spec.vocab, m.top) or t.is_floating_point() or int(t.min()) < 0 or int(t.max()) >= m.experts:
+                        raise ValueError("the routing table holds `top` experts for every token id")
+                    d["table"] = t.to(self.device, torch.int32).contiguous()
+                else:
+                    d["router"] = self._f32(w["router"])
                 d["gu"] = self._act(torch.stack([torch.cat([g, u], dim=0) for g, u, _ in w["experts"]]))
                 d["down"] = self._act(torch.stack([dn for _, _, dn in w["experts"]]))
                 assert d["gu"].shape == (m.experts, 2 * m.ff, self.spec.width)
@@ -532,6 +592,8 @@ class SeqStateModel:
             if l.mixer == "retention":
                 cl.rot_dims, cl.inv_freq, cl.decay = l.rot_dims, p(w["inv_freq"]), p(w["decay"])
                 cl.ret_state = p(cache.ret_state[i])
+                cl.act_qkv, cl.k_scale, cl.gate_act = _QKV_ACTS[l.qkv_act], l.k_scale, _GATE_ACTS[l.gate_act]
+                cl.out_norm_w, cl.norm_parts = p(w.get("out_norm")), l.norm_parts
             elif l.mixer == "cached_attention":
                 cl.kv_heads, cl.attn_mode, cl.gate_kind = l.kv_heads, _ATTN_MODES[l.attn_mode], l.gate_kind
                 cl.values_are_keys, cl.pool, cl.taps, cl.window, cl.scale = int(l.values_are_keys), l.pool, l.taps, l.window, l.scale
@@ -549,6 +611,8 @@ class SeqStateModel:
                 cl.chunk, cl.maps, cl.diff_lambda = l.chunk, l.maps, w.get("diff_lambda", 0.0)
                 cl.head_unit_norm, cl.out_mult = int(l.head_unit_norm), (1.0 - l.diff) if l.maps == 2 else 1.0
                 cl.q_norm_w, cl.k_norm_w = p(w.get("q_norm")), p(w.get("k_norm"))
+                cl.q_norm_all_w, cl.k_norm_all_w, cl.sink = p(w.get("q_norm_all")), p(w.get("k_norm_all")), p(w.get("sink"))
+                cl.v_mix, cl.v_lambda = _V_MIXES[l.v_mix], w.get("v_lambda", 0.0)
             elif l.mixer == "time_mix":
                 cl.mix_mu, cl.decay_rank, cl.w_decay1, cl.w_decay2 = p(w["mu"]), l.decay_rank, p(w["w1"]), p(w["w2"])
                 cl.decay_bias, cl.bonus, cl.out_norm_w = p(w["w0"]), p(w["u"]), p(w["out_norm"])
@@ -568,7 +632,7 @@ class SeqStateModel:
                     p(w["ukT"]), p(w["uv"])
                 cl.w_ukv = p(w["ukv"]) if self.fresh_attention else None
                 cl.ring = p(cache.ring[i])
-                if l.q_rank == 0:
+                if l.form == "prenorm":
                     cl.rope_dim, cl.rot_dims, cl.inv_freq, cl.rot_mag = l.rope_dim, l.rot_dims, p(w["inv_freq"]), l.rot_mag
                     cl.attn_mode, cl.gate_kind, cl.sink = _ATTN_MODES[l.attn_mode], l.gate_kind, p(w.get("sink"))
             cl.w_in, cl.w_o = p(w["w_in"]), p(w["o"])
@@ -584,7 +648,7 @@ class SeqStateModel:
             cl.norm_alpha, cl.norm2_alpha = w.get("norm_alpha", 1.0), w.get("norm2_alpha", 1.0)
             cl.post_norm_w, cl.post_norm2_w = p(w.get("post_norm")), p(w.get("post_norm2"))
             cl.out_scale, cl.out_scale2, cl.residual_mult = p(w.get("ls1")), p(w.get("ls2")), l.residual_mult
-            cl.norm_w = p(w["norm"])
+            cl.norm_w = p(w.get("norm"))
             if l.mixer != "time_mix":
                 cl.shift_w, cl.shift_state = p(w.get("shift")), p(cache.shift[i])
             cl.depth_w = p(w.get("depth"))
@@ -605,13 +669,15 @@ class SeqStateModel:
                 cl.mlp.bias_gu, cl.mlp.bias_down = p(w.get("s_gu_b")), p(w.get("s_down_b"))
                 cl.mlp.w_shared_gate = p(w.get("s_gate"))
                 cl.mlp.route_scale = m.route_scale
+                cl.mlp.route_table = p(w.get("table"))
                 if m.plain:
-                    cl.mlp.plain, cl.mlp.unary = 1, S.UMBS_UNARY_XIELU
-                    cl.mlp.unary_p0, cl.mlp.unary_p1 = w["unary_p"]
+                    cl.mlp.plain, cl.mlp.unary = 1, _PLAIN_ACTS[m.plain]
+                    cl.mlp.unary_p0, cl.mlp.unary_p1 = w.get("unary_p", (0.0, 0.0))
         m = S.Model()
         m.dtype = S.UMBS_BF16 if self.dtype == torch.bfloat16 else S.UMBS_F32
         m.width, m.vocab, m.n_layers, m.norm_groups, m.slots = sp.width, sp.vocab, len(self.runs), sp.norm_groups, cache.slots
         m.norm_eps, m.norm_offset, m.logit_softcap = sp.norm_eps, sp.norm_offset, sp.logit_softcap
+        m.logit_scale = sp.logit_scale
         hw = self.head_weights
         m.embed, m.final_norm, m.head = p(hw["embed"]), p(hw["final_norm"]), p(hw["head"])
         m.embed_scale, m.norm_kind, m.final_norm_b = sp.embed_scale, _NORMS[sp.norm_kind], p(hw.get("final_norm_b"))
