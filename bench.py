@@ -19,6 +19,8 @@ scripted acceptance with the reference's DEFAULT_ACC (random weights make draft 
   kulisun            the latent-attention family with a shared rotated key part and a group-limited router next to Radanex
   subivik            the family of talking / differential attention beside a time-mix memory next to Zedotar at equal size
   ralapel            the family of looped layers, rank-one memories and latent attention next to Zedotar and Kulisun at equal size
+  revudra            the family of blocks without norms in front (windowed, lightning and latent mixers, experts by token id) next to
+                     Kulisun, Radanex and Zedotar at equal size
   static70b_b200tree the default workload on the packaged B200-tuned 16-node tree (sequoia_utils.generate_budget_tree)
 
 A *step* is one speculative-decoding iteration (draft build_tree + target verify + accept + KV gather).  ``value`` =
@@ -76,6 +78,7 @@ WORKLOADS["radanex"] = dict(text="Radanex bf16 vs Llama fp16 at equal width / de
 WORKLOADS["zedotar"] = dict(text="Zedotar bf16 vs Radanex bf16 at equal width / depth: prefill and decode tokens/s, kernel table")
 WORKLOADS["kulisun"] = dict(text="Kulisun bf16 vs Radanex bf16 at equal width / depth: prefill and decode tokens/s, kernel table")
 WORKLOADS["ralapel"] = dict(text="Ralapel bf16 vs Zedotar and Kulisun bf16 at equal width / depth: prefill and decode tokens/s, kernel table")
+WORKLOADS["revudra"] = dict(text="Revudra bf16 vs Kulisun, Radanex and Zedotar bf16 at equal width / depth: prefill and decode tokens/s, kernel table")
 WORKLOADS["subivik"] = dict(text="Subivik bf16 vs Zedotar bf16 at equal width / depth: prefill and decode tokens/s, kernel table")
 E2E_REQUESTS = 8          # per replica (2 for stochastic32k: a 30k-token prefill and PCIe-bound verifies per request)
 
@@ -510,6 +513,9 @@ def main():
     if args.workload == "ralapel":
         from umbrella_b200 import seq_bench
         return seq_bench.run_ralapel(args)
+    if args.workload == "revudra":
+        from umbrella_b200 import seq_bench
+        return seq_bench.run_revudra(args)
     run_ours(args)
 
 

@@ -1,7 +1,7 @@
-"""One prefill step and a few eager decode steps of a synthetic Radanex (or Zedotar, Kulisun, Subivik or Ralapel) model: the program to put under
+"""One prefill step and a few eager decode steps of a synthetic Radanex (or Zedotar, Kulisun, Subivik, Ralapel or Revudra) model: the program to put under
 `ncu --metrics gpu__time_duration.sum` for a launch list of the sequence-state step (small: < 1 GB on the device).
 
-    python scripts/seq_step_once.py [width] [batch] [context] [decode steps] [radanex|zedotar|kulisun|subivik|ralapel]
+    python scripts/seq_step_once.py [width] [batch] [context] [decode steps] [radanex|zedotar|kulisun|subivik|ralapel|revudra]
 """
 import os
 import sys
@@ -24,6 +24,9 @@ elif len(sys.argv) > 5 and sys.argv[5] == "subivik":
 elif len(sys.argv) > 5 and sys.argv[5] == "ralapel":
     from umbrella_b200.models.ralapel import Ralapel as Family, spec_from_config  # noqa: E402
     spec = spec_from_config(seq_bench.ralapel_config(width, 8))
+elif len(sys.argv) > 5 and sys.argv[5] == "revudra":
+    from umbrella_b200.models.revudra import Revudra as Family, spec_from_config  # noqa: E402
+    spec = spec_from_config(seq_bench.revudra_config(width, 8))
 else:
     from umbrella_b200.models.radanex import Radanex as Family, spec_from_config  # noqa: E402
     spec = spec_from_config(seq_bench.radanex_config(width, 8))

@@ -348,3 +348,63 @@ def test_state_cache_of_looped_memories():
     spec.loop = (2, 2, 1)
     with pytest.raises(ValueError):
         SeqStateModel(spec, device="cpu")
+
+
+# ---------------------------------------------------------------------------------------------- the Revudra family
+def test_revudra_config_reader_and_tensor_names():
+    import copy
+    import rev_helpers as U
+    from umbrella_b200.models.revudra import layer_tensor_names, spec_from_config, synth_tensors
+    spec = spec_from_config(U.MIXED)
+    assert (spec.width, spec.vocab, spec.norm_eps, spec.embed_scale, spec.logit_scale, spec.norm_kind) == (72, 101, 1e-5, 3.0, 0.4, "rms")
+    assert all(l.form == "prenorm" and not l.pre_norm and l.post_norm and l.residual_mult == 0.6 and not l.shift and not l.depth_average for l in spec.layers)
+    g, a0, a1, t, a2, g2, a3, t2 = spec.layers
+    assert (g.mixer, g.heads, g.dim, g.vdim, g.qkv_act, g.k_scale, g.out_norm, g.gate_act, g.rot_dims) == ("retention", 5, 11, 14, "silu", 1.0, True, "sigmoid", 0)
+    assert g.decay == U.MIXED["layers"][0]["mixer"]["decay"] and (g.mlp.experts, g.mlp.top, g.mlp.ff, g.mlp.route, g.mlp.act) == (5, 3, 20, "table", "silu")
+    assert (a1.mixer, a1.heads, a1.kv_heads, a1.dim, a1.vdim, a1.window, a1.rot_dims, a1.rot_base) == ("cached_attention", 6, 3, 10, 14, 17, 10, 50.0)
+    assert (a1.attn_mode, a1.learned_sink, a1.gate_kind, a1.qk_norm_all, a1.qk_norm) == ("softmax_sink", True, 2, True, False)
+    assert [l.v_mix for l in spec.layers] == ["", "", "source", "", "mix", "", "mix", ""]
+    assert (a1.mlp.plain, a1.mlp.shared_ff, a1.mlp.experts, a0.mlp, a3.window) == ("relu2", 44, 0, None, 1)
+    assert (t.mixer, t.q_rank, t.kv_rank, t.rope_dim, t.rot_dims, t.rot_pairs, t.gate_kind, t.attn_mode, t.learned_sink, t.window) == \
+        ("latent_attention", 26, 20, 6, 6, "neighbours", 1, "softmax_sink", True, 0)
+    assert (t2.rot_base, g2.mlp, a2.scale) == (1000.0, None, U.MIXED["layers"][4]["mixer"]["scale"])
+
+    def flat(v):
+        return [x for y in v for x in flat(y)] if isinstance(v, (list, tuple)) else [v]
+    tensors = U.random_tensors(U.MIXED)
+    names = {n for i in range(len(spec.layers)) for n in flat(list(layer_tensor_names(spec, i).values()))}
+    # (the first mixing layer's own number is never read)
+    assert names | {"embed", "head", "final.norm", "l2.mix.vmix"} == set(tensors)
+    assert {k: tuple(v.shape) for k, v in synth_tensors(spec, 1).items()} == {k: tuple(v.shape) for k, v in tensors.items() if k != "l2.mix.vmix"}
+    table = synth_tensors(spec, 1)["l0.mlp.table"]
+    assert all(len(set(row)) == 3 and 0 <= min(row) and max(row) < 5 for row in table.tolist())
+    for path, value in ((("layers", 0, "mixer", "decay"), [0.5] * 4), (("layers", 1, "mixer", "kv_heads"), 3), (("layers", 3, "mixer", "rot", "dims"), 8),
+                        (("layers", 1, "mixer", "rot", "dims"), 7), (("layers", 0, "mlp", "router", "top"), 6), (("layers", 0, "mlp", "kind"), "sparse"),
+                        (("layers", 2, "type"), "delta"), (("architecture",), "Ralapel")):
+        bad = copy.deepcopy(U.MIXED)
+        at = bad
+        for k in path[:-1]:
+            at = at[k]
+        at[path[-1]] = value
+        with pytest.raises(ValueError):
+            spec_from_config(bad)
+
+
+def test_revudra_state_cache_and_value_sources():
+    import rev_helpers as U
+    from umbrella_b200.attn.state_cache import SequenceStateCache
+    from umbrella_b200.models.revudra import spec_from_config
+    from umbrella_b200.models.seq_model import SeqStateModel
+    spec = spec_from_config(U.MIXED)
+    c = SequenceStateCache(spec, slots=2, device="cpu", dtype=torch.float32, capacity=24)
+    assert c.ret_state[0].shape == (2, 5, 11, 14) and c.kv_cache[1].shape == (2, 9, 2 * 32) and c.kv_cache[2].shape == (2, 17, 3 * 24)
+    assert c.ring[3].shape == (2, 24, 26) and c.kv_cache[6].shape == (2, 1, 48) and all(t is None for t in c.shift + c.conv_state)
+    c.reserve_length(30)
+    assert c.ring[7].shape == (2, 48, 40) and c.kv_cache[4].shape == (2, 24, 3 * 30)      # windows do not grow
+    SeqStateModel(spec, device="cpu")
+    spec.layers[4].vdim = 10                                          # a layer cannot mix in values of another size
+    with pytest.raises(ValueError):
+        SeqStateModel(spec, device="cpu")
+    spec.layers[4].vdim, spec.layers[2].v_mix = 14, ""                # ... or without a source in front of it
+    with pytest.raises(ValueError):
+        SeqStateModel(spec, device="cpu")

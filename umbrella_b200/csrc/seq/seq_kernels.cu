@@ -157,7 +157,7 @@ __global__ void rotary_table_kernel(const int32_t* __restrict__ tok_pos, const f
 // output in shared memory, and the parts are added in warp order.  TB = 16 (8 for the widest heads, whose staging
 // registers would not fit): a round's serial walk then outlasts the latency of the next round's scattered loads.
 template <int DPT, int kRetTB>
-__global__ void retention_kernel(const float* __restrict__ qkvg, int64_t ld, Batch b, int heads, int dim, int vdim,
+__global__ void __launch_bounds__(DPT == 8 ? 128 : (DPT == 16 ? 256 : 512)) retention_kernel(const float* __restrict__ qkvg, int64_t ld, Batch b, int heads, int dim, int vdim,
                                  int rot_dims, const float* __restrict__ rot_tab, const float* __restrict__ inv_freq,
                                  const float* __restrict__ decay, float* __restrict__ state, float* __restrict__ o_out,
                                  float kscale, int seg_len, int n_seg, int pass, float* __restrict__ seg_state) {

@@ -87,16 +87,20 @@ def group_norm_shift(x, w, shift_w, shift_state, batch: RaggedBatch, groups: int
 
 
 def retention(qkvg, batch: RaggedBatch, heads, dim, vdim, rot_dims, inv_freq, decay, eps, state, dtype=torch.float32,
-              segments: bool = True):
-    """``segments``: give the kernel room to cut few long sequences into segments that run side by side."""
+              segments: bool = True, k_scale: float = 0.0, norm_w=None, norm_parts: int = 1, gate_act: int = S.UMBS_GATE_SILU):
+    """``segments``: give the kernel room to cut few long sequences into segments that run side by side.  ``k_scale`` (0:
+    dim^-1/2), ``norm_w`` (RMS norm over the concatenated heads in ``norm_parts`` parts instead of one per head), ``gate_act``:
+    the options of umbs_retention_ex."""
     T = qkvg.shape[0]
     seg = torch.empty(32 * heads * dim * vdim, dtype=torch.float32, device=qkvg.device) if segments and T >= 128 else None
     o32 = torch.empty((T, heads * vdim), dtype=torch.float32, device=qkvg.device)
     out = torch.empty((T, heads * vdim), dtype=dtype, device=qkvg.device)
     rot = torch.empty((T, max(rot_dims, 1)), dtype=torch.float32, device=qkvg.device)
-    S.check(S.load().umbs_retention(_mode(out), _p(qkvg), qkvg.stride(0), C.byref(batch.c), heads, dim, vdim, rot_dims,
-                                    _p(inv_freq), _p(decay), float(eps), _p(state), _p(o32), _p(rot), _p(seg),
-                                    seg.numel() * 4 if seg is not None else 0, _p(out), _stream()),
+    o = S.RetentionOpts()
+    o.k_scale, o.norm_w, o.norm_parts, o.gate_act = float(k_scale), norm_w.data_ptr() if norm_w is not None else None, norm_parts, gate_act
+    S.check(S.load().umbs_retention_ex(_mode(out), _p(qkvg), qkvg.stride(0), C.byref(batch.c), heads, dim, vdim, rot_dims,
+                                       _p(inv_freq), _p(decay), float(eps), _p(state), _p(o32), _p(rot), _p(seg),
+                                       seg.numel() * 4 if seg is not None else 0, C.byref(o), _p(out), _stream()),
             "retention")
     return out
 
@@ -192,7 +196,7 @@ def attention_prep(proj, bias, batch: RaggedBatch, heads, kv_heads, dim, vdim, r
 
 def cached_attention(q, kv, kv_cache, batch: RaggedBatch, heads, kv_heads, dim, vdim, scale, mode=S.UMBS_ATTN_SOFTMAX,
                      window=0, pool=0, pool_cache=None, head_bias=None, gate=None, gate_per_head=False, append=True,
-                     split=True):
+                     split=True, sink=None):
     """One attention step over the step's kv rows and the slots' caches (pooling the blocks the step completes first and
     appending the step's rows afterwards, as umbs_forward does)."""
     T = q.shape[0]
@@ -202,11 +206,13 @@ def cached_attention(q, kv, kv_cache, batch: RaggedBatch, heads, kv_heads, dim, 
         S.check(lib.umbs_kv_pool(_mode(q), _p(kv), _p(kv_cache), kv_cache.shape[1], _p(pool_cache), pool_cache.shape[1],
                                  C.byref(batch.c), row, pool, _stream()), "kv_pool")
     part = torch.empty(2048 * (vdim + 2), dtype=torch.float32, device=q.device) if split else None
-    S.check(lib.umbs_cached_attention(_mode(q), mode, _p(q), _p(kv), _p(kv_cache), kv_cache.shape[1], _p(pool_cache),
-                                      pool_cache.shape[1] if pool_cache is not None else 0, C.byref(batch.c), heads, kv_heads,
-                                      dim, vdim, window, pool, float(scale), _p(head_bias), _p(gate),
-                                      gate.stride(0) if gate is not None else 0, int(gate_per_head), _p(part),
-                                      part.numel() * 4 if part is not None else 0, _p(out), _stream()), "cached_attention")
+    o = S.AttnOpts()
+    o.sink = sink.data_ptr() if sink is not None else None
+    S.check(lib.umbs_cached_attention_ex(_mode(q), mode, _p(q), _p(kv), _p(kv_cache), kv_cache.shape[1], _p(pool_cache),
+                                         pool_cache.shape[1] if pool_cache is not None else 0, C.byref(batch.c), heads, kv_heads,
+                                         dim, vdim, window, pool, float(scale), _p(head_bias), _p(gate),
+                                         gate.stride(0) if gate is not None else 0, int(gate_per_head), C.byref(o), _p(part),
+                                         part.numel() * 4 if part is not None else 0, _p(out), _stream()), "cached_attention")
     if append:
         S.check(lib.umbs_ring_append(_mode(q), _p(kv), _p(kv_cache), kv_cache.shape[1], C.byref(batch.c), row, _stream()),
                 "ring_append")
@@ -302,7 +308,7 @@ def latent_attention_shared(q_abs, c, ring, batch: RaggedBatch, heads, kv_rank, 
 
 
 def window_attention_shared(q, k, k_shared, v, batch: RaggedBatch, heads: int, scale: float, window: int = 0, sink=None,
-                            use_sink: bool = True, gate=None):
+                            use_sink: bool = True, gate=None, gate_per_head: bool = False):
     """q [T, heads (dim + shared)], k [T, heads dim], k_shared [T, shared], v [T, heads vdim] (row-strided views are fine)
     -> [T, heads vdim]: attention among the step's own tokens with a key part all heads share, a sink and an output gate."""
     T = q.shape[0]
@@ -310,12 +316,12 @@ def window_attention_shared(q, k, k_shared, v, batch: RaggedBatch, heads: int, s
     dim, vdim = k.shape[1] // heads, v.shape[1] // heads
     assert q.shape[1] == heads * (dim + sd)
     out = torch.empty((T, heads * vdim), dtype=q.dtype, device=q.device)
-    S.check(S.load().umbs_window_attention_ex(_mode(q), _p(q), q.stride(0), _p(k), k.stride(0), _p(k_shared),
-                                              k_shared.stride(0) if k_shared is not None else 0, sd, _p(v), v.stride(0),
-                                              C.byref(batch.c), heads, dim, vdim, window, float(scale),
-                                              S.UMBS_ATTN_SOFTMAX_SINK if use_sink else S.UMBS_ATTN_SOFTMAX, _p(sink), _p(gate),
-                                              gate.stride(0) if gate is not None else 0, _p(out), heads * vdim, _stream()),
-            "window_attention_ex")
+    S.check(S.load().umbs_window_attention_gated(_mode(q), _p(q), q.stride(0), _p(k), k.stride(0), _p(k_shared),
+                                                 k_shared.stride(0) if k_shared is not None else 0, sd, _p(v), v.stride(0),
+                                                 C.byref(batch.c), heads, dim, vdim, window, float(scale),
+                                                 S.UMBS_ATTN_SOFTMAX_SINK if use_sink else S.UMBS_ATTN_SOFTMAX, _p(sink), _p(gate),
+                                                 gate.stride(0) if gate is not None else 0, int(gate_per_head), _p(out), heads * vdim,
+                                                 _stream()), "window_attention_gated")
     return out
 
 
@@ -437,13 +443,13 @@ def time_mix(proj, decay_raw, decay_bias, bonus, batch: RaggedBatch, heads, dim,
     return out
 
 
-def gemm_unary(a: torch.Tensor, w: torch.Tensor, unary: int, p0: float = 0.0, p1: float = 0.0, out_f32: bool = False):
-    """unary(a [M, K] x w [N, K]^T): UMBS_UNARY_TANH or UMBS_UNARY_XIELU with its two coefficients."""
+def gemm_unary(a: torch.Tensor, w: torch.Tensor, unary: int, p0: float = 0.0, p1: float = 0.0, out_f32: bool = False, cols: int = 0):
+    """unary(a [M, K] x w [N, K]^T): UMBS_UNARY_* (with its two coefficients, where it has any), on the first ``cols`` columns (0: all)."""
     assert w.dtype == a.dtype and a.stride(-1) == 1 and w.is_contiguous()
     out = torch.empty((a.shape[0], w.shape[0]), dtype=torch.float32 if out_f32 else a.dtype, device=a.device)
-    S.check(S.load().umbs_gemm_unary(_mode(a), _p(a), a.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0,
-                                     int(out_f32), a.shape[0], w.shape[0], w.shape[1], 1, None, unary, float(p0), float(p1),
-                                     _stream()), "gemm_unary")
+    S.check(S.load().umbs_gemm_unary_cols(_mode(a), _p(a), a.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0,
+                                          int(out_f32), a.shape[0], w.shape[0], w.shape[1], 1, None, unary, float(p0), float(p1), cols,
+                                          _stream()), "gemm_unary_cols")
     return out
 
 
@@ -476,13 +482,16 @@ def add_post_norm(x, delta, post_w, w, eps: float, dtype=torch.float32, rows=Non
     return (y, copy) if want_copy else y
 
 
-def add_rows(x, out, delta=None, post_w=None, eps: float = 0.0):
-    """x [n, width] fp32 += delta (through an RMS norm with ``post_w`` if given); out[:, :width] = x in out's dtype (out may have
-    a longer row)."""
+def add_rows(x, out, delta=None, post_w=None, eps: float = 0.0, mult: float = 1.0, pair_out=None, sel_w=None, pair_pos=None):
+    """x [n, width] fp32 += mult * (delta, or the routed experts' rows; through an RMS norm with ``post_w`` if given);
+    out[:, :width] = x in out's dtype (out may have a longer row)."""
     d = None
-    if delta is not None:
+    if delta is not None or pair_out is not None:
         d = S.Delta()
-        d.delta, d.mult, d.delta_mult, d.norm_w = delta.data_ptr(), 1.0, 1.0, post_w.data_ptr() if post_w is not None else None
+        d.mult, d.delta_mult = float(mult), 1.0
+        d.delta, d.norm_w, d.pair_out, d.sel_w, d.pair_pos = (t.data_ptr() if t is not None else None
+                                                              for t in (delta, post_w, pair_out, sel_w, pair_pos))
+        d.top = sel_w.shape[1] if sel_w is not None else 0
     S.check(S.load().umbs_add_rows(_mode(out), _p(x), C.byref(d) if d is not None else None, x.shape[0], x.shape[1], float(eps), _p(out),
                                    out.stride(0), None, _stream()), "add_rows")
     return out
@@ -529,9 +538,89 @@ def memory_run(qkv, gates, kq, mem, batch: RaggedBatch):
     return o
 
 
-def gated_norm(o, gate, parts: int, w, gate_first: bool, eps: float, dtype=torch.float32):
-    """unit(o silu(gate)) * w (``gate_first``) or unit(o) * w * silu(gate), unit RMS over each of ``parts`` equal parts of a row."""
+def gated_norm(o, gate, parts: int, w, gate_first: bool, eps: float, dtype=torch.float32, gate_act: int = S.UMBS_GATE_SILU):
+    """unit(o act(gate)) * w (``gate_first``) or unit(o) * w * act(gate), unit RMS over each of ``parts`` equal parts of a row; act =
+    silu or (UMBS_GATE_SIGMOID) sigmoid."""
     out = torch.empty(o.shape, dtype=dtype, device=o.device)
-    S.check(S.load().umbs_gated_norm(_mode(out), _p(o), _p(gate), gate.stride(0), o.shape[0], o.shape[1], parts, _p(w), w.numel(),
-                                     int(gate_first), float(eps), _p(out), _stream()), "gated_norm")
+    S.check(S.load().umbs_gated_norm_ex(_mode(out), _p(o), _p(gate), gate.stride(0), o.shape[0], o.shape[1], parts, _p(w), w.numel(),
+                                        int(gate_first), gate_act, float(eps), _p(out), _stream()), "gated_norm")
     return out
+
+
+# ---------------------------------------------------------------------------------------------- blocks that read the stream, routing by token id
+def embedding_rows(ids, table, scale: float = 1.0):
+    """table[ids] * scale -> (fp32 [n, width], the same in the table's dtype)."""
+    y = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    y2 = torch.empty((ids.numel(), table.shape[1]), dtype=table.dtype, device=table.device)
+    S.check(S.load().umbs_embedding_rows(_mode(table), _p(ids), None, _p(table), float(scale), None, _p(y), _p(y2), ids.numel(),
+                                         table.shape[1], _stream()), "embedding_rows")
+    return y, y2
+
+
+def attention_prep_rows(proj, batch: RaggedBatch, heads, kv_heads, dim, vdim, rot_dims, inv_freq, q_norm_all=None, k_norm_all=None,
+                        eps=1e-6, v_mix: int = S.UMBS_VMIX_NONE, v_lambda: float = 0.0, v_source=None, dtype=torch.float32):
+    """proj fp32 [T, q | k | v | ...] -> (q, kv) as ``dtype``: RMS norms over the whole query and the whole key row, rotary
+    positions, values written to or mixed with ``v_source`` (fp32 [T, kv_heads vdim], UMBS_VMIX_*)."""
+    T = proj.shape[0]
+    q = torch.empty((T, heads * dim), dtype=dtype, device=proj.device)
+    kv = torch.empty((T, kv_heads * (dim + vdim)), dtype=dtype, device=proj.device)
+    o = S.PrepOpts()
+    o.q_norm_all_w, o.k_norm_all_w, o.v_source = (t.data_ptr() if t is not None else None for t in (q_norm_all, k_norm_all, v_source))
+    o.v_mix, o.v_lambda = v_mix, float(v_lambda)
+    S.check(S.load().umbs_attention_prep_opts(_mode(q), _p(proj), proj.stride(0), None, C.byref(batch.c), heads, kv_heads, dim, vdim, 0, 1,
+                                              None, None, 0, rot_dims, _p(inv_freq), 1.0, 1, None, None, float(eps), C.byref(o), _p(q),
+                                              _p(kv), _stream()), "attention_prep_opts")
+    return q, kv
+
+
+def latent_low_prep(proj, batch: RaggedBatch, q_rank, q_norm, kv_rank, kv_norm, rope_dim, rot_dims, inv_freq, eps, rot_mag=1.0,
+                    dtype=torch.float32):
+    """proj fp32 [T, query latent | latent | shared key part | ...] -> (normed query latent [T, q_rank], c [T, kv_rank + rope_dim])."""
+    T = proj.shape[0]
+    cq = torch.empty((T, q_rank), dtype=dtype, device=proj.device)
+    c = torch.empty((T, kv_rank + rope_dim), dtype=dtype, device=proj.device)
+    p = S.LatentPrep()
+    p.dq, p.ld_dq, p.q_rank, p.q_norm, p.cq = proj.data_ptr(), proj.stride(0), q_rank, q_norm.data_ptr(), cq.data_ptr()
+    p.low, p.ld_low, p.kv_rank, p.kv_norm, p.c = proj.data_ptr() + 4 * q_rank, proj.stride(0), kv_rank, kv_norm.data_ptr(), c.data_ptr()
+    p.rope_dim, p.rot_dims, p.inv_freq, p.rot_mag, p.eps = rope_dim, rot_dims, inv_freq.data_ptr(), float(rot_mag), float(eps)
+    S.check(S.load().umbs_latent_prep_parts(_mode(cq), C.byref(p), C.byref(batch.c), _stream()), "latent_prep_parts")
+    return cq, c
+
+
+def latent_query_turn(qsrc, batch: RaggedBatch, heads, dim, rope_dim, kv_rank, rot_dims, inv_freq, rot_mag=1.0, dtype=torch.float32):
+    """qsrc fp32 [T, heads (dim + rope_dim)] -> (q as ``dtype`` with every head's rope part turned, q_abs fp32 [T, heads, kv_rank +
+    rope_dim] holding the turned parts behind room for the product with the key up-projection)."""
+    T, KD = qsrc.shape[0], kv_rank + rope_dim
+    q = torch.empty((T, heads * (dim + rope_dim)), dtype=dtype, device=qsrc.device)
+    q_abs = torch.zeros((T, heads, KD), dtype=torch.float32, device=qsrc.device)
+    p = S.LatentPrep()
+    p.qsrc, p.ld_q, p.heads, p.dim, p.q = qsrc.data_ptr(), qsrc.stride(0), heads, dim, q.data_ptr()
+    p.q_rot, p.ld_qrot = q_abs.data_ptr() + 4 * kv_rank, KD
+    p.rope_dim, p.rot_dims, p.inv_freq, p.rot_mag = rope_dim, rot_dims, inv_freq.data_ptr(), float(rot_mag)
+    S.check(S.load().umbs_latent_prep_parts(_mode(q), C.byref(p), C.byref(batch.c), _stream()), "latent_prep_parts")
+    return q, q_abs
+
+
+def gemm_head_gate(a, w, out_gate, groups: int, n: int, k: int):
+    """a [M, groups k] x w [groups, n, k] -> [M, groups n], group g's columns times sigmoid(out_gate[row, g]) (fp32, row-strided)."""
+    out = torch.empty((a.shape[0], groups * n), dtype=a.dtype, device=a.device)
+    S.check(S.load().umbs_gemm_head_gate(_mode(a), _p(a), a.stride(0), k, _p(w), k, n * k, _p(out), out.stride(0), n, 0, a.shape[0], n, k,
+                                         groups, _p(out_gate), out_gate.stride(0), _stream()), "gemm_head_gate")
+    return out
+
+
+def table_route(ids, tables, outs=None):
+    """Routing by token id.  ``tables``: [(table int32 [vocab, top], experts)] -> per layer (sel_w, grp_off, pair_tok, pair_pos), one
+    launch for all of them; ``outs``: an earlier call's result of the same sizes to write over."""
+    n, dev, given, outs = ids.numel(), ids.device, outs, []
+    arr = (S.TableRoute * len(tables))()
+    for i, (r, (table, experts)) in enumerate(zip(arr, tables)):
+        top = table.shape[1]
+        o = given[i] if given is not None else \
+            (torch.empty((n, top), dtype=torch.float32, device=dev), torch.empty(experts + 1, dtype=torch.int32, device=dev),
+             torch.empty(n * top, dtype=torch.int32, device=dev), torch.empty(n * top, dtype=torch.int32, device=dev))
+        r.table, r.experts, r.top = table.data_ptr(), experts, top
+        r.sel_w, r.grp_off, r.pair_tok, r.pair_pos = (t.data_ptr() for t in o)
+        outs.append(o)
+    S.check(S.load().umbs_table_route(_p(ids), n, arr, len(tables), _stream()), "table_route")
+    return outs

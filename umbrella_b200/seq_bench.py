@@ -1003,3 +1003,211 @@ def run_ralapel(args):
                        "l2": "whole-model runs stream more than L2 per step; kernel table flushes L2 between runs"},
             "sizes": sizes, "kernels": table}
     print(json.dumps(line))
+
+
+def revudra_config(width: int, layers: int = 8) -> dict:
+    """A Revudra config with the layer sizes of a model of this width: windowed attention (heads of 128 over the width, a quarter as
+    many key / value heads, 1024 tokens), lightning memories (heads of 128 x 128), latent attention of Kulisun's sizes with a
+    query latent of 3/8 of the width, attention again; the first layer's feed-forward dense, the others 2 of 8 experts as wide
+    as the model (the active width and about the weights of Kulisun's 2 of 16 beside a shared expert)."""
+    heads = max(2, width // 128)
+    att = dict(type="attention", mixer=dict(heads=heads, kv_heads=max(1, heads // 4), dim=128, vdim=128, scale=128 ** -0.5, v_mix=True,
+                                            mask=dict(size=1024), rot=dict(dims=64, base=1e6)))
+    lig = dict(type="lightning", mixer=dict(heads=heads, dim=128, vdim=128, decay=[1 - 2.0 ** (-3 - (6 * h) // heads) for h in range(heads)]))
+    lat = dict(type="latent_attention", mixer=dict(heads=heads, dim=128, rot_dim=64, vdim=128, q_rank=3 * width // 8, kv_rank=width // 4,
+                                                   scale=192 ** -0.5, rot=dict(base=1e4, dims=64)))
+    dense, moe = dict(kind="dense", ff=2 * width), dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=width))
+    return dict(architecture="Revudra", width=width, vocab=32768, norm=dict(eps=1e-6), embedding=dict(scale=10.0), residual_mult=0.8,
+                logit_scale=0.5, layers=[dict((att, lig, lat, att)[i % 4], mlp=moe if i else dense) for i in range(layers)])
+
+
+def bench_revudra(width, layers, device, prompt, ctx, batches, timer):
+    from .models.revudra import Revudra, spec_from_config
+    spec = spec_from_config(revudra_config(width, layers))
+    m = Revudra(spec, device=device, dtype=torch.bfloat16, slots=max(batches), max_tokens=prompt + ctx)
+    return bench_seq_model(m, spec, prompt, ctx, batches, timer)
+
+
+def kernel_table_revudra(vm, km, rm, zm, device, timer, T=4096):
+    """Device time of each Revudra mechanism at prefill size (one sequence of T tokens) and at decode size (8 and 64 sequences
+    behind 512 tokens), with its roofline fractions, and the like kernels of the Kulisun, Radanex and Zedotar paths measured the
+    same way in the same run (``like`` names the pairing)."""
+    from . import _lib_seq as S, ops_seq as Q
+    hbm, tflops, how = _peaks()
+    sp, W = vm.spec, vm.spec.width
+    fp32_peak = 148 * 128 * 2 * 1.965e-3
+    rows = []
+
+    def add(name, ms, nbytes=0, flops=0, like=None, flops32=0):
+        r = dict(kernel=name, ms=round(ms, 4))
+        if flops32:
+            r["fp32_tflops"], r["frac_of_fp32_fma_peak"] = round(flops32 / ms / 1e9, 2), round(flops32 / ms / 1e9 / fp32_peak, 3)
+        if flops:
+            r["tflops"], r["frac_of_bf16_peak"] = round(flops / ms / 1e9, 1), round(flops / ms / 1e9 / tflops, 3)
+        if nbytes:
+            r["gb_s"], r["frac_of_hbm_peak"] = round(nbytes / ms / 1e6, 1), round(nbytes / ms / 1e6 / hbm, 3)
+        if like:
+            r["like"] = like
+        rows.append(r)
+    pick = lambda spec, kind, **kw: next(i for i, l in enumerate(spec.layers) if l.mixer == kind and all(getattr(l, k) == v for k, v in kw.items()))
+    ksp, rsp, zsp = km.spec, rm.spec, zm.spec
+    ai, gi, li = pick(sp, "cached_attention", v_mix="mix"), pick(sp, "retention"), pick(sp, "latent_attention")
+    ri, zi = pick(rsp, "retention"), pick(zsp, "cached_attention", window=1024)
+    za = pick(zsp, "cached_attention", taps=4)
+    att, lig, lat, ret, zat, klat = sp.layers[ai], sp.layers[gi], sp.layers[li], rsp.layers[ri], zsp.layers[zi], ksp.layers[1]
+    aw, gw, lw, dw = vm.weights[ai], vm.weights[gi], vm.weights[li], vm.weights[0]
+    rw, zw, kw, kd = rm.weights[ri], zm.weights[zi], km.weights[1], km.weights[0]
+    bf = dict(dtype=torch.bfloat16, device=device)
+    ctx = 512
+    for m in (vm, km, zm):
+        m.cache.reserve_length(T)
+    g = torch.Generator().manual_seed(1)
+    for n, tag in ((T, f"prefill T={T}"), (8, "decode T=8"), (64, "decode T=64")):
+        nseq = 1 if n == T else n
+        per = n // nseq
+        pos0 = 0 if n == T else ctx
+        batch = Q.RaggedBatch([(s, per, pos0, 0) for s in range(nseq)], device)
+        ids = torch.randint(0, sp.vocab, (n,), generator=g).to(torch.int32).to(device)
+        x, d, h = torch.randn(n, W, device=device), torch.randn(n, W, device=device), torch.randn(n, W, **bf)
+        # routing: every routed layer of the model in one launch, against one router
+        f, kf = lig.mlp, klat.mlp
+        tables = [(w["table"], l.mlp.experts) for l, w in zip(sp.layers, vm.weights) if "table" in w]
+        routes = Q.table_route(ids, tables)
+        ms = timer(lambda: Q.table_route(ids, tables, routes))
+        add(f"routing by token id, {len(tables)} layers in one launch ({tag})", ms, nbytes=len(tables) * n * f.top * (4 + 4 + 4 + 4), like="kulisun router")
+        ms = timer(lambda: Q.moe_route_ex(h, kw["router"], kf.top, S.UMBS_ROUTE_SIGMOID_GROUPS, kf.groups, kf.keep))
+        add(f"kulisun router + expert sort, one layer ({tag})", ms, nbytes=n * W * 2)
+        sel_w, grp_off, pair_tok, pair_pos = routes[0]
+        ksel, kgo, kpt, kpp, _ = Q.moe_route_ex(h, kw["router"], kf.top, S.UMBS_ROUTE_SIGMOID_GROUPS, kf.groups, kf.keep)
+        # norms behind the blocks
+        pair_out, sg, buf = torch.randn(n * f.top, W, device=device), torch.rand(n, device=device), torch.empty(n, W, **bf)
+        ms = timer(lambda: Q.add_rows(x, buf, d, aw["post_norm"], sp.norm_eps, mult=0.8))
+        add(f"norm behind the block + residual add + rows for the next block ({tag})", ms, nbytes=n * W * (4 + 4 + 4 + 2), like="kulisun residual add + layer norm")
+        ms = timer(lambda: Q.add_rows(x, buf, None, aw["post_norm2"], sp.norm_eps, mult=0.8, pair_out=pair_out, sel_w=sel_w, pair_pos=pair_pos))
+        add(f"norm behind {f.top} routed outputs + residual add + rows ({tag})", ms, nbytes=n * W * (4 + 4 + 2 + 4 * f.top),
+            like="kulisun residual add of routed")
+        ms = timer(lambda: Q.add_norm(x, kd["norm"], kd["norm_b"], ksp.norm_eps, dtype=torch.bfloat16, delta=d, scale=kd["ls1"], mult=0.7))
+        add(f"kulisun residual add + layer norm ({tag})", ms, nbytes=n * W * (4 + 4 + 4 + 2))
+        ms = timer(lambda: Q.add_norm(x, kd["norm"], kd["norm_b"], ksp.norm_eps, dtype=torch.bfloat16, pair_out=pair_out, sel_w=ksel, pair_pos=kpp,
+                                      shared=d, shared_gate=sg, scale=kd["ls1"], mult=0.7))
+        add(f"kulisun residual add of routed + gated shared outputs + layer norm ({tag})", ms, nbytes=n * W * (4 + 4 + 4 + 2 + 4 * kf.top))
+        # products
+        for name, w, cols, like in (("gemm lightning in-projection + silu on q, k, v", gw["w_in"], gw["w_in"].shape[0] - lig.heads * lig.vdim, "radanex gemm in-projection"),
+                                    ("radanex gemm in-projection", rw["w_in"], 0, None)):
+            ms = timer(lambda: Q.gemm_unary(h, w, S.UMBS_UNARY_SILU if cols else 0, out_f32=True, cols=cols))
+            add(f"{name} [{n} x {W}] x [{w.shape[0]} x {W}] ({tag})", ms, nbytes=w.numel() * 2 + n * W * 2 + n * w.shape[0] * 4,
+                flops=2 * n * W * w.shape[0], like=like)
+        up, kgu = dw["s_gu"], kd["s_gu"]
+        ms = timer(lambda: Q.gemm_unary(h, up, S.UMBS_UNARY_RELU2))
+        add(f"gemm dense up + squared relu [{n} x {W}] x [{up.shape[0]} x {W}] ({tag})", ms, nbytes=up.numel() * 2 + n * W * 2 + n * up.shape[0] * 2,
+            flops=2 * n * up.numel(), like="kulisun gemm dense down")
+        kdn, hf = kd["s_down"], torch.randn(n, kd["s_down"].shape[1], **bf)
+        ms = timer(lambda: Q.gemm(hf, kdn, out_f32=True))
+        add(f"kulisun gemm dense down [{n} x {kdn.shape[1]}] x [{W} x {kdn.shape[1]}] ({tag})", ms, nbytes=kdn.numel() * 2 + hf.numel() * 2 + n * W * 4,
+            flops=2 * n * kdn.numel())
+        ms = timer(lambda: Q.gemm_ex(h, kgu, act=S.UMBS_ACT_SILU, bias=kd["s_gu_b"]))
+        add(f"kulisun gemm dense gate|up + bias + silu [{n} x {W}] x [{kgu.shape[0]} x {W}] ({tag})", ms, nbytes=kgu.numel() * 2 + n * W * 2 + n * kgu.shape[0],
+            flops=2 * n * kgu.numel())
+        for who, ff, w, go, pt in (("", f, gw, grp_off, pair_tok), ("kulisun ", kf, kw, kgo, kpt)):
+            ms = timer(lambda: Q.gemm(h, w["gu"], groups=ff.experts, n=ff.ff, dual=S.UMBS_ACT_SILU, grp_off=go, row_src=pt, rows=n * ff.top, max_rows=n))
+            touched = min(ff.experts, n * ff.top)
+            add(f"{who}gemm routed gate|up + silu, {ff.experts} experts top {ff.top} of {ff.ff} ({tag})", ms,
+                nbytes=touched * 2 * ff.ff * W * 2 + n * W * 2 + n * ff.top * ff.ff * 2, flops=2 * n * ff.top * W * 2 * ff.ff,
+                like=None if who else "kulisun gemm routed")
+        # lightning beside retention
+        for who, l, w, model, i, kwargs in (("", lig, gw, vm, gi, dict(k_scale=1.0, norm_w=gw["out_norm"], gate_act=S.UMBS_GATE_SIGMOID)), ("radanex ", ret, rw, rm, ri, {})):
+            ld = 2 * l.heads * (l.dim + l.vdim)
+            qkvg = torch.randn(n, ld, device=device)
+            state = model.cache.ret_state[i]
+            ms = timer(lambda: Q.retention(qkvg, batch, l.heads, l.dim, l.vdim, l.rot_dims, w["inv_freq"], w["decay"], 1e-6, state, torch.bfloat16, **kwargs))
+            what = "radanex retention: rotary + recurrence + unit norm + gate" if who else "lightning: recurrence + norm over the heads + gate"
+            add(f"{what}, fp32, {l.heads} heads of {l.dim} x {l.vdim} ({tag})", ms, flops32=4 * n * l.heads * l.dim * l.vdim,
+                nbytes=n * ld * 4 + n * l.heads * l.vdim * (4 + 4 + 2) + nseq * l.heads * l.dim * l.vdim * 8, like=None if who else "radanex retention")
+        # windowed attention beside Zedotar's
+        H, G, D, V = att.heads, att.kv_heads, att.dim, att.vdim
+        ld = (H + G) * D + G * V + H * V
+        proj, vs = torch.randn(n, ld, device=device), torch.randn(n, G * V, device=device)
+        ms = timer(lambda: Q.attention_prep_rows(proj, batch, H, G, D, V, att.rot_dims, aw["inv_freq"], aw["q_norm_all"], aw["k_norm_all"], 1e-6,
+                                                 S.UMBS_VMIX_MIX, 0.3, vs, torch.bfloat16))
+        add(f"attention prep: norms over q and k + rotary + mixed values ({tag})", ms, nbytes=n * (H * D + G * (D + V)) * (4 + 2) + n * G * V * 4,
+            like="zedotar attention prep")
+        zl, zaw = zsp.layers[za], zm.weights[za]
+        zpr, zcs = torch.randn(n, (zl.heads + zl.kv_heads) * zl.dim + zl.heads * zl.vdim, device=device), zm.cache.conv_state[za]
+        ms = timer(lambda: Q.attention_prep(zpr, zaw.get("bias_in"), batch, zl.heads, zl.kv_heads, zl.dim, zl.dim, zl.rot_dims, zaw["inv_freq"], zl.rot_mag,
+                                            True, zl.taps, zaw["conv_w"], zcs, torch.bfloat16))
+        add(f"zedotar attention prep: convolution + rotary ({tag})", ms, nbytes=n * (zl.heads + zl.kv_heads) * zl.dim * 4 + n * (zl.heads + 2 * zl.kv_heads) * zl.dim * 2)
+        gate = proj[:, (H + G) * D + G * V:]
+        for who, l, w, cache, kwargs in (("", att, aw, vm.cache.kv_cache[ai], dict(mode=S.UMBS_ATTN_SOFTMAX_SINK, sink=aw["sink"], gate=gate)),
+                                         ("zedotar ", zat, zw, zm.cache.kv_cache[zi], dict(pool=zat.pool, pool_cache=zm.cache.pool_cache[zi]))):
+            q, kv = torch.randn(n, l.heads * l.dim, **bf), torch.randn(n, l.kv_heads * (l.dim + l.vdim), **bf)
+            keys = sum(min(p + 1, l.window) + (max(0, (p - l.window + 1)) // l.pool if l.pool else 0) for p in range(pos0, pos0 + per)) * nseq
+            ms = timer(lambda: Q.cached_attention(q, kv, cache, batch, l.heads, l.kv_heads, l.dim, l.vdim, l.scale, window=l.window, append=False, **kwargs))
+            what = "zedotar attention, window + pooled blocks" if who else "attention, window, sink, gate"
+            add(f"{what}, {l.window} tokens, fp32 scores ({tag})", ms, flops32=2 * keys * l.heads * (l.dim + l.vdim),
+                nbytes=n * (2 * l.heads * l.dim + l.kv_heads * (l.dim + l.vdim)) * 2 + (0 if n == T else keys * l.kv_heads * (l.dim + l.vdim) * 2)
+                + (0 if who else n * H * V * 4), like=None if who else "zedotar attention, window")
+        # latent attention beside Kulisun's
+        H, D, Rt, R, V = lat.heads, lat.dim, lat.rope_dim, lat.kv_rank, lat.vdim
+        KD, hdq = R + Rt, H * (D + Rt)
+        low, q32 = torch.randn(n, lat.q_rank + KD + H, device=device), torch.randn(n, hdq, device=device)
+
+        def both():
+            Q.latent_low_prep(low, batch, lat.q_rank, lw["q_norm"], R, lw["kv_norm"], Rt, lat.rot_dims, lw["inv_freq"], 1e-6, dtype=torch.bfloat16)
+            Q.latent_query_turn(q32, batch, H, D, Rt, R, lat.rot_dims, lw["inv_freq"], dtype=torch.bfloat16)
+        add(f"latent norms + rotary, both launches ({tag})", timer(both), nbytes=n * (hdq + KD + lat.q_rank) * (4 + 2) + n * H * Rt * 4, like="kulisun latent norm")
+        kproj = torch.randn(n, hdq + KD + H * V, device=device)
+        ms = timer(lambda: Q.latent_prep(kproj, batch, H, D, Rt, R, kw["kv_norm"], 1e-6, klat.rot_dims, kw["inv_freq"], klat.rot_mag, torch.bfloat16))
+        add(f"kulisun latent norm + rotary ({tag})", ms, nbytes=n * (hdq + KD) * (4 + 2) + n * H * Rt * 4)
+        keys = sum(p + 1 for p in range(pos0, pos0 + per)) * nseq
+        uv = lw["uv"].view(H, V, R)
+        for who, w, gt, per_head, ring in (("", lw, low[:, lat.q_rank + KD:], True, vm.cache.ring[li]), ("kulisun ", kw, kproj[:, hdq + KD:], False, km.cache.ring[1])):
+            like = (lambda s: None) if who else (lambda s: "kulisun " + s)
+            if n == T:
+                q, kvh, ks = torch.randn(n, hdq, **bf), torch.randn(n, H * (D + V), **bf), torch.randn(n, KD, **bf)
+                ms = timer(lambda: Q.window_attention_shared(q, kvh[:, :H * D], ks[:, R:], kvh[:, H * D:], batch, H, lat.scale, sink=w["sink"], gate=gt,
+                                                             gate_per_head=per_head))
+                add(f"{who}attention over per-head keys + shared rotated part, causal, sink, gate, fp32 scores ({tag})", ms,
+                    nbytes=n * (hdq + H * (D + V) + Rt + H * V) * 2 + n * H * (1 if per_head else V) * 4, flops32=2 * keys * H * (D + Rt + V),
+                    like=like("attention over per-head keys"))
+            else:
+                qa, c, o_lat = torch.randn(n, H, KD, device=device), torch.randn(n, KD, **bf), torch.randn(n, H * R, **bf)
+                ms = timer(lambda: Q.latent_attention_shared(qa, c, ring, batch, H, R, Rt, lat.scale, sink=w["sink"], append=False))
+                add(f"{who}latent attention over [latent | shared part] keys, causal, sink, fp32 scores ({tag})", ms,
+                    nbytes=n * H * (KD * 4 + R * 2) + keys * KD * 2, flops32=2 * keys * H * (KD + R), like=like("latent attention"))
+                ms = timer((lambda: Q.gemm_head_gate(o_lat, uv, gt, H, V, R)) if per_head else
+                           (lambda: Q.gemm_ex(o_lat, uv, groups=H, a_goff=R, c_goff=V, n=V, k=R, out_gate=gt, gate_goff=V)))
+                add(f"{who}gemm value up-projection per head + gate ({tag})", ms, nbytes=n * H * R * 2 + H * V * R * 2 + n * H * V * 2 + n * H * (1 if per_head else V) * 4,
+                    flops=2 * n * H * V * R, like=like("gemm value up-projection"))
+    return rows, how
+
+
+def run_revudra(args):
+    from . import _lib_seq
+    device = "cuda:0"
+    timer = Timer(device)
+    hbm, tflops, how = _peaks()
+    sizes, table = [], None
+    launches0 = _lib_seq.load().umbs_launch_count()
+    for width in (1024, 2048):
+        layers, prompt, ctx = 8, 2048, 512
+        models, row = {}, {"width": width, "layers": layers}
+        for name, bench in (("revudra", bench_revudra), ("kulisun", bench_kulisun), ("radanex", bench_radanex), ("zedotar", bench_zedotar)):
+            models[name], r = bench(width, layers, device, prompt, ctx, (1, 8, 64), timer)
+            row[f"{name}_bf16"] = {n: round(v, 3) for n, v in r.items()}
+        sizes.append(row)
+        if width == 2048:
+            table, _ = kernel_table_revudra(models["revudra"], models["kulisun"], models["radanex"], models["zedotar"], device, timer)
+        models.clear()
+        torch.cuda.empty_cache()
+    launches = _lib_seq.load().umbs_launch_count() - launches0
+    head = sizes[-1]["revudra_bf16"]
+    line = {"metric": "decode tokens/sec at batch 64 (Revudra bf16, width 2048, 8 layers, synthetic weights)",
+            "value": head["decode_b64_tok_s"], "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16",
+            "data": "synthetic", "vs_baseline": None, "gpu_launches": int(launches),
+            "config": {"name": "revudra", "workload": "prefill 1 x 2048 and 4 x 2048 tokens; decode at batch 1 / 8 / 64 behind a "
+                       "512-token context; Kulisun bf16 (the closest family: latent attention with sinks and gates, routed experts of the same "
+                       "active width), Radanex bf16 (retention) and Zedotar bf16 (windowed attention) of the same width and depth beside it",
+                       "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": how},
+                       "l2": "whole-model runs stream more than L2 per step; kernel table flushes L2 between runs"},
+            "sizes": sizes, "kernels": table}
+    print(json.dumps(line))
