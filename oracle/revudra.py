@@ -56,7 +56,7 @@ def rotate_pairs(x, base, first=0):
 
 
 def visible(n, window):
-    """[n, n] bool: row i sees j with 0 <= i - j < window (window 0: every j <= i)."""
+    """[n, n] bool: the last ``window`` keys up to the row itself (window 0: all of them)."""
     d = torch.arange(n)[:, None] - torch.arange(n)[None, :]
     return (d >= 0) & ((d < window) if window else torch.ones_like(d, dtype=torch.bool))
 

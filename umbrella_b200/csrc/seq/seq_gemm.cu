@@ -290,18 +290,13 @@ __global__ void __launch_bounds__(32 * SK_WARPS) gemm_skinny_kernel(GemmArgs a) 
         arow[m] = A + (int64_t)(a.row_src ? a.row_src[p] : p) * a.lda;
     }
     float acc[SK_ROWS][MT] = {};
-    uint4 wv[SK_ROWS];                     // the next step's weights are on their way while this step's are used
-#pragma unroll
-    for (int i = 0; i < SK_ROWS; ++i)
-        wv[i] = lane * 8 < a.K ? __ldg(reinterpret_cast<const uint4*>(wrow[i] + lane * 8)) : make_uint4(0, 0, 0, 0);
     for (int k = lane * 8; k < a.K; k += 256) {
+        uint4 wv[SK_ROWS];
+#pragma unroll
+        for (int i = 0; i < SK_ROWS; ++i) wv[i] = __ldg(reinterpret_cast<const uint4*>(wrow[i] + k));
         float wf[SK_ROWS][8];
 #pragma unroll
         for (int i = 0; i < SK_ROWS; ++i) bf16x8_to_f32(wv[i], wf[i]);
-        if (k + 256 < a.K) {
-#pragma unroll
-            for (int i = 0; i < SK_ROWS; ++i) wv[i] = __ldg(reinterpret_cast<const uint4*>(wrow[i] + k + 256));
-        }
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
             float af[8];

@@ -744,8 +744,20 @@ __global__ void __launch_bounds__(1024) table_route_kernel(const int32_t* __rest
     int32_t* next = cnt + E;
     for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
     __syncthreads();
+    // a thread's first KEEP choices stay in registers for the second walk, their loads all in flight together
+    constexpr int KEEP = 8;
+    auto choice = [&](int i) -> int { const int t = i / r.top; return r.table[(int64_t)ids[t] * r.top + (i - t * r.top)]; };
+    int kept[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        kept[j] = i < pairs ? choice(i) : -1;
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j)
+        if (kept[j] >= 0) atomicAdd(cnt + kept[j], 1);
 #pragma unroll 4
-    for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(cnt + r.table[(int64_t)ids[i / r.top] * r.top + i % r.top], 1);
+    for (int i = threadIdx.x + KEEP * blockDim.x; i < pairs; i += blockDim.x) atomicAdd(cnt + choice(i), 1);
     __syncthreads();
     int base = 0;                                    // exclusive sums over the experts, a block's width at a time
     for (int e0 = 0; e0 < E; e0 += blockDim.x) {
@@ -770,13 +782,17 @@ __global__ void __launch_bounds__(1024) table_route_kernel(const int32_t* __rest
     }
     if (threadIdx.x == 0) r.grp_off[E] = base;
     const float wgt = 1.f / (float)r.top;
-#pragma unroll 4
-    for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-        const int t = i / r.top, p = atomicAdd(next + r.table[(int64_t)ids[t] * r.top + (i - t * r.top)], 1);
-        r.pair_tok[p] = t;
+    auto hand_out = [&](int i, int e) {
+        const int p = atomicAdd(next + e, 1);
+        r.pair_tok[p] = i / r.top;
         r.pair_pos[i] = p;
         r.sel_w[i] = wgt;
-    }
+    };
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j)
+        if (kept[j] >= 0) hand_out(threadIdx.x + j * blockDim.x, kept[j]);
+#pragma unroll 4
+    for (int i = threadIdx.x + KEEP * blockDim.x; i < pairs; i += blockDim.x) hand_out(i, choice(i));
 }
 
 // One warp per token: g[t] = sigmoid(w . h[t]).
